@@ -7,10 +7,11 @@ page-major): every execution of a mixer that keeps keys and values owns two pool
 64 x head_dim block.
 
 Executions are sorted into *groups* by what they need to keep: all keys (window 0) or
-only the last ``window`` keys.  Each group has its own page pool and its own block
+only the last ``window`` keys, with or without the first ``keep_first``.  Each group has its own page pool and its own block
 table per request; inside a group the same page id indexes every member's pools, since
 members grow in step.  A request's pages go back to the pool when it ends, and in a
-window group also as soon as the window has passed them.
+window group also as soon as the window has passed them (all but those of kept first
+positions).
 
 Fixed-size state (the short convolution's rolling inputs here; any recurrent state in
 general) lives in *slots*: every such execution owns one ``[num_slots][...]`` tensor in the
@@ -100,6 +101,7 @@ class PageGroup:
     pool: PagePool
     members: List[int] = field(default_factory=list)      # schedule positions
     tables: Dict[Hashable, List[int]] = field(default_factory=dict)   # logical page -> id or -1
+    keep_first: int = 0                       # positions from 0 on that stay readable in a window group
 
     def first_needed_page(self, length: int) -> int:
         """Lowest logical page a query at position ``length`` (the next one) still reads."""
@@ -132,7 +134,7 @@ class CacheManager:
         self._serial: Dict[Hashable, int] = {}
         self._admissions = 0
         self.slots_high_water = 0
-        by_window: Dict[int, int] = {}
+        by_window: Dict[Tuple[int, int], int] = {}
         self._fixed_specs: Dict[int, FixedState] = {}
         for position, spec in enumerate(state_specs):
             members = spec if isinstance(spec, tuple) else (() if spec is None else (spec,))
@@ -144,10 +146,11 @@ class CacheManager:
             cache = LayerCache(spec=spec)
             if paged:
                 kv = paged[0]
-                if kv.window not in by_window:
-                    by_window[kv.window] = len(self.groups)
-                    self.groups.append(PageGroup(kv.window, PagePool(self.num_pages)))
-                cache.group = by_window[kv.window]
+                kept = kv.keep_first if kv.window > 0 else 0
+                if (kv.window, kept) not in by_window:
+                    by_window[kv.window, kept] = len(self.groups)
+                    self.groups.append(PageGroup(kv.window, PagePool(self.num_pages), keep_first=kept))
+                cache.group = by_window[kv.window, kept]
                 self.groups[cache.group].members.append(position)
                 if device is not None:
                     shape = (self.num_pages, kv.n_kv_heads, PAGE_SIZE, kv.head_dim)
@@ -235,7 +238,7 @@ class CacheManager:
         for group in self.groups:
             table = group.tables[request]
             first = group.first_needed_page(self._length[request])
-            for logical in range(min(first, len(table))):
+            for logical in range(-(-group.keep_first // PAGE_SIZE), min(first, len(table))):
                 if table[logical] >= 0:
                     group.pool.release(table[logical])
                     table[logical] = -1
@@ -388,7 +391,7 @@ class CacheManager:
     def stats(self) -> dict:
         return {
             "page_size": PAGE_SIZE,
-            "groups": [{"window": g.window, "layers": len(g.members), "pages": g.pool.num_pages,
+            "groups": [{"window": g.window, "keep_first": g.keep_first, "layers": len(g.members), "pages": g.pool.num_pages,
                         "pages_in_use": g.pool.n_used, "pages_high_water": g.pool.high_water}
                        for g in self.groups],
             "slots": self.num_slots, "slots_in_use": len(self._slot_of),

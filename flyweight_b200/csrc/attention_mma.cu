@@ -169,7 +169,7 @@ __device__ __forceinline__ void pv_tile(float (&o)[HD / 8][4], const float (&p)[
 template <int HD, int NT>
 __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&o)[HD / 8][4], float (&m)[2],
                                                float (&l)[2], int key_base, const int (&lo)[2],
-                                               const int (&hi)[2], float scale, float softcap, int lane) {
+                                               const int (&hi)[2], int keep, float scale, float softcap, int lane) {
     const int t = lane & 3;
     // capped scores: cap * tanh(score / cap), in base 2 like the scale (which has log2(e) folded in)
     const float cap_pre = softcap > 0.0f ? scale / (softcap * LOG2E) : 0.0f, cap_post = softcap * LOG2E;
@@ -181,7 +181,7 @@ __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&o)[HD 
             const int key = key_base + n * 8 + 2 * t + (j & 1);
             const int h = j >> 1;
             const float capped = softcap > 0.0f ? cap_post * fwb::tanh_fast_f32(s[n][j] * cap_pre) : s[n][j] * scale;
-            const float v = (key >= lo[h] && key <= hi[h]) ? capped : -INFINITY;   // scale has log2(e) folded in
+            const float v = ((key >= lo[h] || key < keep) && key <= hi[h]) ? capped : -INFINITY;   // scale has log2(e) folded in
             s[n][j] = v;
             mx[h] = fmaxf(mx[h], v);
         }
@@ -247,7 +247,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
                          const int* __restrict__ tile_tok0, const int* __restrict__ block_table,
                          int max_pages, __nv_bfloat16* __restrict__ out, int nh, int nkv, int group,
                          int tokens_per_tile, int window, float scale, const float* __restrict__ sink,
-                         int pool_nkv, float softcap) {
+                         int pool_nkv, float softcap, int keep) {
     fwb::pdl_entry();
     extern __shared__ __align__(16) uint8_t smem_raw[];
     __nv_bfloat16* smem = reinterpret_cast<__nv_bfloat16*>(smem_raw);
@@ -280,10 +280,11 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
     uint32_t qf[HD / 16][4];
     load_q<HD>(qf, qrow[0], qrow[1], lane);
 
-    // keys this CTA walks: from the lowest key any row may see to the position of its last token
+    // keys this CTA walks: from the lowest key any row may see to the position of its last token, behind
+    // the tiles of kept first positions
     const int pos_first = positions[tok0], pos_last = positions[tok0 + n_tok - 1];
     const int lo_block = fwb::first_visible_key(pos_first, window);
-    const int tile_begin = lo_block / KEYS, tile_end = pos_last / KEYS + 1;
+    const KeyTiles walk = fwb::key_tiles(lo_block, pos_last, keep, KEYS);
 
     float o[HD / 8][4];
 #pragma unroll
@@ -313,11 +314,11 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
         load_tile<HD>(stage_k(s), stage_v(s), k_pool, v_pool, src, !same);
         cp_async_commit();
     };
-    issue(tile_begin, 0);
-    for (int tile = tile_begin; tile < tile_end; ++tile) {
-        const int s = (tile - tile_begin) & 1;
-        if (tile + 1 < tile_end) {
-            issue(tile + 1, s ^ 1);
+    issue(walk.at(0), 0);
+    for (int step = 0; step < walk.count; ++step) {
+        const int s = step & 1, tile = walk.at(step);
+        if (step + 1 < walk.count) {
+            issue(walk.at(step + 1), s ^ 1);
             cp_async_wait<1>();
         } else {
             cp_async_wait<0>();
@@ -332,7 +333,7 @@ attention_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat1
         if (warp_hi >= tile * KEYS) {
             float sc[8][4];
             qk_tile<HD, 8>(sc, qf, stage_k(s), 0, lane);
-            softmax_update<HD, 8>(sc, o, m, l, tile * KEYS, lo, hi, scale, softcap, lane);
+            softmax_update<HD, 8>(sc, o, m, l, tile * KEYS, lo, hi, keep, scale, softcap, lane);
             pv_tile<HD, 8>(o, sc, stage_v(s), 0, lane);
         }
         __syncthreads();                                    // the stage may be overwritten next
@@ -355,6 +356,7 @@ struct FusedQkv {
     const float* sink;           // [nh] or null: a score per head that joins the softmax denominator (no value)
     int pool_nkv;                // heads of the pools; 0: nkv (else several groups of query heads share a pool head)
     float softcap;               // > 0: score <- softcap * tanh(score / softcap) behind the scale
+    int keep;                    // > 0: the first `keep` positions stay visible beside the window
     const __nv_bfloat16* qkv;    // [T][(nh + 2 nkv_in) HD]; null: `q` holds finished queries
     const float* wq;             // [HD] head-norm weights (unused when !use_norm)
     const float* wk;
@@ -445,10 +447,13 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     const int pos = positions[tok];
     const int lo_key = fwb::first_visible_key(pos, window);
     const int* table = block_table + (size_t)tok_seg[tok] * max_pages;
-    const int first_tile = lo_key / KEYS, last_tile = pos / KEYS;
-    const int tile_begin = first_tile + split * tiles_per_split;
-    int tile_end = tile_begin + tiles_per_split;
-    if (tile_end > last_tile + 1) tile_end = last_tile + 1;
+    // a slice is a run of steps of the walk over the token's tiles (kept first tiles, then the window's);
+    // the walk's last step is the tile of the token itself
+    const KeyTiles walk = fwb::key_tiles(lo_key, pos, fused.keep, KEYS);
+    const int last_step = walk.count - 1;
+    const int step_begin = split * tiles_per_split;
+    int step_end = step_begin + tiles_per_split;
+    if (step_end > walk.count) step_end = walk.count;
     const int pool_nkv = fused.pool_nkv > 0 ? fused.pool_nkv : nkv;
     const int pool_kvh = (int)((long)kvh * pool_nkv / nkv);
 
@@ -471,9 +476,10 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         }
         __syncthreads();
     }
-    auto issue = [&](int tile, int s) {
+    auto issue = [&](int step, int s) {
+        const int tile = walk.at(step);
         if (TMA) {
-            if (threadIdx.x == 0 && tile < tile_end) {
+            if (threadIdx.x == 0 && step < step_end) {
                 // the stage was read (and, in a token's last tile, cleared) through ordinary loads and stores
                 asm volatile("fence.proxy.async.shared::cta;" ::: "memory");
                 tc5::mbar_expect_tx(&full_bar[s], (same ? 1 : 2) * TILE * 2);
@@ -486,7 +492,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
             }
             return;
         }
-        if (tile < tile_end) {
+        if (step < step_end) {
             const size_t src = ((size_t)table[tile] * pool_nkv + pool_kvh) * KEYS * HD;
             load_tile<HD>(stage_k(s), stage_v(s), k_pool, v_pool, src, !same);
         }
@@ -495,18 +501,18 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
     // every tile but the token's own last one was written by earlier steps: those among the first
     // DECODE_STAGES - 1 are fetched before the wait for the previous kernel
     int issued = 0;
-    while (issued < DECODE_STAGES - 1 && tile_begin + issued < tile_end && tile_begin + issued < last_tile) {
-        issue(tile_begin + issued, issued);
+    while (issued < DECODE_STAGES - 1 && step_begin + issued < step_end && step_begin + issued < last_step) {
+        issue(step_begin + issued, issued);
         ++issued;
     }
     fwb::pdl_wait();
 
     constexpr bool fuse = FUSED;
     // the slice that holds the token's own position also norms, turns and stores its key and value
-    const bool owns_token = fuse && fused.nkv_in > 0 && last_tile >= tile_begin && last_tile < tile_end;
+    const bool owns_token = fuse && fused.nkv_in > 0 && last_step >= step_begin && last_step < step_end;
     if constexpr (fuse) {
         fused_heads<HD>(fused, tok, pos, kvh, nh, nkv, group, owns_token,
-                        owns_token ? (((size_t)table[last_tile] * nkv + kvh) * KEYS + (size_t)(pos % KEYS)) * HD : 0,
+                        owns_token ? (((size_t)table[pos / KEYS] * nkv + kvh) * KEYS + (size_t)(pos % KEYS)) * HD : 0,
                         own_q, own_kv);
         __syncthreads();
     }
@@ -537,20 +543,20 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         }
     }
 
-    for (; issued < DECODE_STAGES - 1; ++issued) issue(tile_begin + issued, issued);
-    for (int tile = tile_begin; tile < tile_end; ++tile) {
-        const int s = (tile - tile_begin) % DECODE_STAGES;
+    for (; issued < DECODE_STAGES - 1; ++issued) issue(step_begin + issued, issued);
+    for (int step = step_begin; step < step_end; ++step) {
+        const int s = (step - step_begin) % DECODE_STAGES, tile = walk.at(step);
         // the slot this tile's successor-but-two goes to was read in the iteration before this one
-        issue(tile + DECODE_STAGES - 1, (tile - tile_begin + DECODE_STAGES - 1) % DECODE_STAGES);
+        issue(step + DECODE_STAGES - 1, (step - step_begin + DECODE_STAGES - 1) % DECODE_STAGES);
         if (TMA) {
             // the tile's bytes have landed when its barrier's phase completes; a thread that has
             // seen that may read them
-            tc5::mbar_wait(&full_bar[s], (uint32_t)((tile - tile_begin) / DECODE_STAGES) & 1u, &abort_flag, 21, status);
+            tc5::mbar_wait(&full_bar[s], (uint32_t)((step - step_begin) / DECODE_STAGES) & 1u, &abort_flag, 21, status);
         } else {
             cp_async_wait<(DEEP ? decode_stages<HD>() : 2) - 1>();
             __syncthreads();
         }
-        if (tile == last_tile && (owns_token || pos - tile * KEYS + 1 < KEYS)) {
+        if (step == last_step && (owns_token || pos - tile * KEYS + 1 < KEYS)) {
             if (owns_token && threadIdx.x < 2 * (HD / 8)) {
                 // the page row of the token itself: what this CTA has just computed (the copy in the
                 // pool may or may not have been seen by the tile's load)
@@ -564,7 +570,7 @@ attention_decode_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_
         }
         float sc[2][4];                                     // this warp's 16 keys of the tile
         qk_tile<HD, 2, TMA>(sc, qf, stage_k(s), warp * 16, lane);
-        softmax_update<HD, 2>(sc, o, m, l, tile * KEYS + warp * 16, lo, hi, scale, fused.softcap, lane);
+        softmax_update<HD, 2>(sc, o, m, l, tile * KEYS + warp * 16, lo, hi, fused.keep, scale, fused.softcap, lane);
         pv_tile<HD, 2, TMA>(o, sc, stage_v(s), warp * 16, lane);
         __syncthreads();
     }
@@ -716,7 +722,7 @@ template <int HD>
 int launch_prefill(const void* q, const void* k_pool, const void* v_pool, const int* positions,
                    const int* seg_start, const int* tile_seg, const int* tile_tok0, const int* block_table,
                    int max_pages, void* out, int n_tiles, int nh, int nkv, int tokens_per_tile, int window,
-                   float scale, const float* sink, int pool_nkv, float softcap, cudaStream_t stream) {
+                   float scale, const float* sink, int pool_nkv, float softcap, int keep, cudaStream_t stream) {
     auto kernel = attention_prefill_kernel<HD>;
     int st = opt_in_smem(kernel, Smem<HD>::BYTES);
     if (st != FWB_OK) return st;
@@ -724,7 +730,7 @@ int launch_prefill(const void* q, const void* k_pool, const void* v_pool, const 
     fwb::pdl(kernel, dim3(n_tiles, nkv), WARPS * 32, Smem<HD>::BYTES, stream)(
         (const bf*)q, (const bf*)k_pool, (const bf*)v_pool, positions, seg_start, tile_seg, tile_tok0,
         block_table, max_pages, (bf*)out, nh, nkv, nh / nkv, tokens_per_tile, window, scale * LOG2E, sink,
-        pool_nkv > 0 ? pool_nkv : nkv, softcap);
+        pool_nkv > 0 ? pool_nkv : nkv, softcap, keep);
     return fwb_launch_status();
 }
 
@@ -864,13 +870,15 @@ bool shape_ok(int nh, int nkv, int hd, int page_size) {
 // nkv, nkv counts groups of nh / nkv query heads and group i reads pool head i * pool_nkv / nkv
 // (one latent row per token shared by every head: pool_nkv = 1).  v_pool may be k_pool.
 // softcap > 0: score <- softcap * tanh(score / softcap) behind the scale (the sink is not capped).
+// keep > 0 (with a sliding window): the first `keep` positions stay visible beside the window.
 FWB_API int fwb_attention_prefill_mma_capped(const void* q, const void* k_pool, const void* v_pool,
                                              const int* positions, const int* seg_start, const int* tile_seg,
                                              const int* tile_tok0, const int* block_table, int max_pages,
                                              int page_size, void* out, int n_tiles, int nh, int nkv, int hd,
                                              int tokens_per_tile, int window, float scale, const float* sink,
-                                             int pool_nkv, float softcap, cudaStream_t stream) {
+                                             int pool_nkv, float softcap, int keep, cudaStream_t stream) {
     if (n_tiles <= 0) return FWB_OK;
+    if (keep < 0 || (keep > 0 && window <= 0)) return FWB_BAD_ARGUMENT;
     if (!(softcap >= 0.0f)) return FWB_BAD_ARGUMENT;
     if (!q || !k_pool || !v_pool || !positions || !seg_start || !tile_seg || !tile_tok0 || !block_table || !out)
         return FWB_BAD_ARGUMENT;
@@ -879,7 +887,7 @@ FWB_API int fwb_attention_prefill_mma_capped(const void* q, const void* k_pool, 
     if (tokens_per_tile < 1 || tokens_per_tile * (nh / nkv) > 64) return FWB_BAD_ARGUMENT;
 #define CALL(HD)                                                                                          \
     launch_prefill<HD>(q, k_pool, v_pool, positions, seg_start, tile_seg, tile_tok0, block_table, max_pages, \
-                       out, n_tiles, nh, nkv, tokens_per_tile, window, scale, sink, pool_nkv, softcap, stream)
+                       out, n_tiles, nh, nkv, tokens_per_tile, window, scale, sink, pool_nkv, softcap, keep, stream)
     FWB_HD_SWITCH(hd, CALL)
 #undef CALL
 }
@@ -892,7 +900,7 @@ FWB_API int fwb_attention_prefill_mma_sink(const void* q, const void* k_pool, co
                                            int pool_nkv, cudaStream_t stream) {
     return fwb_attention_prefill_mma_capped(q, k_pool, v_pool, positions, seg_start, tile_seg, tile_tok0, block_table,
                                             max_pages, page_size, out, n_tiles, nh, nkv, hd, tokens_per_tile, window,
-                                            scale, sink, pool_nkv, 0.0f, stream);
+                                            scale, sink, pool_nkv, 0.0f, 0, stream);
 }
 
 FWB_API int fwb_attention_prefill_mma(const void* q, const void* k_pool, const void* v_pool,
@@ -907,7 +915,7 @@ FWB_API int fwb_attention_prefill_mma(const void* q, const void* k_pool, const v
     if (tokens_per_tile < 1 || tokens_per_tile * (nh / nkv) > 64) return FWB_BAD_ARGUMENT;
 #define CALL(HD)                                                                                          \
     launch_prefill<HD>(q, k_pool, v_pool, positions, seg_start, tile_seg, tile_tok0, block_table, max_pages, \
-                       out, n_tiles, nh, nkv, tokens_per_tile, window, scale, nullptr, 0, 0.0f, stream)
+                       out, n_tiles, nh, nkv, tokens_per_tile, window, scale, nullptr, 0, 0.0f, 0, stream)
     FWB_HD_SWITCH(hd, CALL)
 #undef CALL
 }
@@ -922,8 +930,10 @@ FWB_API int fwb_attention_decode_mma_capped(const void* q, const void* k_pool, c
                                             int max_pages, int page_size, int num_pages, void* out, float* part_o,
                                             float* part_ml, int T, int nh, int nkv, int hd, int splits,
                                             int tiles_per_split, int window, float scale, int merge_in_cluster,
-                                            const float* sink, int pool_nkv, float softcap, cudaStream_t stream) {
+                                            const float* sink, int pool_nkv, float softcap, int keep,
+                                            cudaStream_t stream) {
     if (T <= 0) return FWB_OK;
+    if (keep < 0 || (keep > 0 && window <= 0)) return FWB_BAD_ARGUMENT;
     if (!(softcap >= 0.0f)) return FWB_BAD_ARGUMENT;
     if (!q || !k_pool || !v_pool || !positions || !tok_seg || !block_table || !out) return FWB_BAD_ARGUMENT;
     if (!shape_ok(nh, nkv, hd, page_size) || T > 65535) return FWB_UNSUPPORTED;
@@ -935,6 +945,7 @@ FWB_API int fwb_attention_decode_mma_capped(const void* q, const void* k_pool, c
     fused.sink = sink;
     fused.pool_nkv = pool_nkv;
     fused.softcap = softcap;
+    fused.keep = keep;
 #define CALL(HD)                                                                                          \
     launch_decode<HD>(q, k_pool, v_pool, positions, tok_seg, block_table, max_pages, num_pages, out, part_o,  \
                       part_ml, T, nh, nkv, splits, tiles_per_split, window, scale, in_cluster, fused, stream)
@@ -951,7 +962,7 @@ FWB_API int fwb_attention_decode_mma_sink(const void* q, const void* k_pool, con
                                           const float* sink, int pool_nkv, cudaStream_t stream) {
     return fwb_attention_decode_mma_capped(q, k_pool, v_pool, positions, tok_seg, block_table, max_pages, page_size,
                                            num_pages, out, part_o, part_ml, T, nh, nkv, hd, splits, tiles_per_split,
-                                           window, scale, merge_in_cluster, sink, pool_nkv, 0.0f, stream);
+                                           window, scale, merge_in_cluster, sink, pool_nkv, 0.0f, 0, stream);
 }
 
 FWB_API int fwb_attention_decode_mma(const void* q, const void* k_pool, const void* v_pool,
@@ -990,8 +1001,7 @@ FWB_API int fwb_attention_decode_fused(const void* qkv, int nkv_in, const float*
     const bool in_cluster = merge_in_cluster != 0 && splits <= 8;
     if (splits < 1 || tiles_per_split < 1 || (splits > 1 && !in_cluster && (!part_o || !part_ml))) return FWB_BAD_ARGUMENT;
     FusedQkv fused;
-    fused.sink = nullptr;
-    fused.pool_nkv = 0;
+    memset(&fused, 0, sizeof(fused));
     fused.qkv = static_cast<const __nv_bfloat16*>(qkv);
     fused.wq = wq;
     fused.wk = wk;

@@ -1,7 +1,8 @@
 // Causal grouped-query attention over the paged cache, plain SIMT, fp32 arithmetic.
 //
 // One block per (query token, KV head).  The block walks the keys that the token may
-// see, lo..pos (lo = max(0, pos-window+1) with a window, else 0), in tiles of 32
+// see, lo..pos (lo = max(0, pos-window+1) with a window, else 0; with `keep` also the
+// positions below it) in tiles of 32
 // positions that start at multiples of 32, stages each K and V tile in shared memory
 // once, and lets its warps run an online softmax for the query heads of that KV head.
 // A tile never straddles a page (the page size is a multiple of 32).  The walk and the
@@ -28,7 +29,7 @@ attention_simt_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_pool,
                       const TC* __restrict__ v_pool, const int* __restrict__ positions,
                       const int* __restrict__ tok_seg, const int* __restrict__ block_table,
                       int max_pages, int page_size, TO* __restrict__ out, int nh, int nkv, int hd,
-                      int window, float scale, const float* __restrict__ sink, float softcap) {
+                      int window, float scale, const float* __restrict__ sink, float softcap, int keep) {
     fwb::pdl_entry();
     extern __shared__ float smem[];
     const int group = nh / nkv;
@@ -60,7 +61,9 @@ attention_simt_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_pool,
     }
     const float inv_cap = softcap > 0.0f ? 1.0f / softcap : 0.0f;
 
-    for (int base = (lo / TILE) * TILE; base <= pos; base += TILE) {
+    const KeyTiles walk = fwb::key_tiles(lo, pos, keep, TILE);
+    for (int tile = 0; tile < walk.count; ++tile) {
+        const int base = walk.at(tile) * TILE;
         __syncthreads();
         const int page = table[base / page_size];
         const size_t src = (((size_t)page * nkv + kvh) * page_size + (base % page_size)) * hd;
@@ -73,7 +76,7 @@ attention_simt_kernel(const TQ* __restrict__ q, const TC* __restrict__ k_pool,
         }
         __syncthreads();
         const int kpos = base + lane;
-        const bool seen = kpos >= lo && kpos <= pos;
+        const bool seen = (kpos >= lo || kpos < keep) && kpos <= pos;
 #pragma unroll
         for (int a = 0; a < MAX_HPW; ++a) {
             const int g = warp + a * WARPS;
@@ -131,13 +134,15 @@ FWB_API int fwb_attention_simt(const void* q, int q_bf16, const void* k_pool, co
 
 // The general form.  sink: fp32 [nh] or null -- a score per head (not scaled, not capped) that joins the
 // row's softmax denominator and has no value.  softcap > 0: score <- softcap * tanh(score / softcap)
-// behind the scale.
+// behind the scale.  keep > 0 (with a sliding window): the sequence's first `keep` positions stay visible
+// however far the window has moved on.
 FWB_API int fwb_attention_simt_sink(const void* q, int q_bf16, const void* k_pool, const void* v_pool,
                                     int cache_bf16, const int* positions, const int* tok_seg,
                                     const int* block_table, int max_pages, int page_size, void* out,
                                     int out_bf16, int T, int nh, int nkv, int hd, int window, float scale,
-                                    const float* sink, float softcap, cudaStream_t stream) {
+                                    const float* sink, float softcap, int keep, cudaStream_t stream) {
     if (T <= 0) return FWB_OK;
+    if (keep < 0 || (keep > 0 && window <= 0)) return FWB_BAD_ARGUMENT;
     if (!q || !k_pool || !v_pool || !positions || !tok_seg || !block_table || !out)
         return FWB_BAD_ARGUMENT;
     if (nh <= 0 || nkv <= 0 || nh % nkv != 0 || hd <= 0 || max_pages <= 0) return FWB_BAD_ARGUMENT;
@@ -159,7 +164,7 @@ FWB_API int fwb_attention_simt_sink(const void* q, int q_bf16, const void* k_poo
         fwb::pdl(kernel, grid, WARPS * 32, smem, stream)((const TQ*)q, (const TC*)k_pool,               \
                                                    (const TC*)v_pool, positions, tok_seg,         \
                                                    block_table, max_pages, page_size, (TO*)out,   \
-                                                   nh, nkv, hd, window, scale, sink, softcap);    \
+                                                   nh, nkv, hd, window, scale, sink, softcap, keep); \
     } while (0)
     if (!q_bf16 && !cache_bf16 && !out_bf16) FWB_ATTN(float, float, float);
     else if (q_bf16 && cache_bf16 && out_bf16) FWB_ATTN(bf, bf, bf);
@@ -175,5 +180,5 @@ FWB_API int fwb_attention_simt(const void* q, int q_bf16, const void* k_pool, co
                                cudaStream_t stream) {
     return fwb_attention_simt_sink(q, q_bf16, k_pool, v_pool, cache_bf16, positions, tok_seg, block_table,
                                    max_pages, page_size, out, out_bf16, T, nh, nkv, hd, window, scale, nullptr,
-                                   0.0f, stream);
+                                   0.0f, 0, stream);
 }

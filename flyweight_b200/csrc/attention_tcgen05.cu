@@ -81,6 +81,7 @@ struct AttnParams {
     const float* sink;           // [nh] or null: a score per head (not scaled) in the softmax denominator, no value
     float cap_pre, cap_unit;     // capped scores: raw <- cap_unit * tanh(raw * cap_pre), cap_pre = scale / cap,
                                  // cap_unit = cap / scale, so that the scale that follows gives cap * tanh(score / cap); 0: off
+    int keep;                    // > 0: the first `keep` positions stay visible beside the window
     int* status;
 };
 
@@ -100,7 +101,8 @@ __device__ __forceinline__ float ex2(float x) {
 
 // One work item: a row tile (up to 128 / group tokens of one segment) and a KV head.
 struct Item {
-    int tok0, kvh, rows, pos_first, pos_last, tile_begin, n_tiles;
+    int tok0, kvh, rows, pos_first, pos_last, n_tiles;
+    KeyTiles walk;               // the key tiles of the item: kept first tiles, then the window's
     const int* table;
 };
 
@@ -116,8 +118,8 @@ __device__ __forceinline__ Item load_item(const AttnParams& prm, int w) {
     it.pos_first = prm.positions[it.tok0];
     it.pos_last = prm.positions[it.tok0 + n_tok - 1];
     const int lo_block = fwb::first_visible_key(it.pos_first, prm.window);
-    it.tile_begin = lo_block / KEYS;
-    it.n_tiles = it.pos_last / KEYS + 1 - it.tile_begin;
+    it.walk = fwb::key_tiles(lo_block, it.pos_last, prm.keep, KEYS);
+    it.n_tiles = it.walk.count;
     it.table = prm.block_table + (size_t)seg * prm.max_pages;
     return it;
 }
@@ -210,13 +212,13 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
                     const bool has_k = t < item.n_tiles, has_v = t >= LEAD;
                     mbar_expect_tx(&full[s], ((has_k ? 1 : 0) + (has_v ? 1 : 0)) * L::KV_BYTES);
                     if (has_k) {
-                        const int row = (item.table[item.tile_begin + t] * prm.nkv + item.kvh) * KEYS;
+                        const int row = (item.table[item.walk.at(t)] * prm.nkv + item.kvh) * KEYS;
 #pragma unroll
                         for (int b = 0; b < L::BOXES; ++b)
                             tma_load_2d(k_s + (size_t)s * L::KV_BYTES + b * L::KV_BOX, &map_k, &full[s], b * 64, row);
                     }
                     if (has_v) {
-                        const int row = (item.table[item.tile_begin + t - LEAD] * prm.nkv + item.kvh) * KEYS;
+                        const int row = (item.table[item.walk.at(t - LEAD)] * prm.nkv + item.kvh) * KEYS;
 #pragma unroll
                         for (int b = 0; b < L::BOXES; ++b)
                             tma_load_2d(v_s + (size_t)s * L::KV_BYTES + b * L::KV_BOX, &map_v, &full[s], b * 64, row);
@@ -324,7 +326,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
             // the highest lower bound of the keys any row of this item may see
             const int lo_max = fwb::first_visible_key(item.pos_last, prm.window);
             for (int j = 0; j < item.n_tiles; ++j) {
-                const int g = g0 + j, key0 = (item.tile_begin + j) * KEYS, buf = g & 1;
+                const int g = g0 + j, key0 = item.walk.at(j) * KEYS, buf = g & 1;
                 ok = mbar_wait(&s_ready[buf], (g >> 1) & 1, abort_flag, 16, prm.status);
                 ok = __all_sync(0xffffffffu, ok);          // tcgen05.ld needs the whole warp
                 if (!ok) break;
@@ -337,12 +339,12 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
                     for (int i = 0; i < KEYS; ++i) sc[i] = prm.cap_unit * fwb::tanh_fast_f32(sc[i] * prm.cap_pre);
                 }
                 // a tile every row sees whole needs no mask (rows without a token are never stored)
-                const bool whole = key0 >= lo_max && key0 + KEYS - 1 <= item.pos_first;
+                const bool whole = (key0 >= lo_max || key0 + KEYS <= prm.keep) && key0 + KEYS - 1 <= item.pos_first;
                 if (!whole) {
 #pragma unroll
                     for (int i = 0; i < KEYS; ++i) {
                         const int key = key0 + i;
-                        sc[i] = (key >= lo && key <= hi) ? sc[i] : -INFINITY;
+                        sc[i] = ((key >= lo || key < prm.keep) && key <= hi) ? sc[i] : -INFINITY;
                     }
                 }
                 // four interleaved chains each for the maximum and the sum: a fixed order, a quarter of the latency
@@ -498,7 +500,7 @@ FWB_API int fwb_attention_prefill_tcgen05_capped(const void* q, const void* k_po
                                                  const int* tile_tok0, const int* block_table, int max_pages,
                                                  int page_size, int num_pages, void* out, int n_tiles, int nh,
                                                  int nkv, int hd, int tokens_per_tile, int window, float scale,
-                                                 const float* sink, float softcap, cudaStream_t stream);
+                                                 const float* sink, float softcap, int keep, cudaStream_t stream);
 
 FWB_API int fwb_attention_prefill_tcgen05_sink(const void* q, const void* k_pool, const void* v_pool,
                                                const int* positions, const int* seg_start, const int* tile_seg,
@@ -508,18 +510,20 @@ FWB_API int fwb_attention_prefill_tcgen05_sink(const void* q, const void* k_pool
                                                const float* sink, cudaStream_t stream) {
     return fwb_attention_prefill_tcgen05_capped(q, k_pool, v_pool, positions, seg_start, tile_seg, tile_tok0,
                                                 block_table, max_pages, page_size, num_pages, out, n_tiles, nh, nkv,
-                                                hd, tokens_per_tile, window, scale, sink, 0.0f, stream);
+                                                hd, tokens_per_tile, window, scale, sink, 0.0f, 0, stream);
 }
 
 // The general form.  softcap > 0: score <- softcap * tanh(score / softcap) behind the scale (the sink is
 // not capped); a scale of 0 with a cap is refused (every score would be 0: not worth a form of its own).
+// keep > 0 (with a sliding window): the first `keep` positions stay visible beside the window.
 FWB_API int fwb_attention_prefill_tcgen05_capped(const void* q, const void* k_pool, const void* v_pool,
                                                  const int* positions, const int* seg_start, const int* tile_seg,
                                                  const int* tile_tok0, const int* block_table, int max_pages,
                                                  int page_size, int num_pages, void* out, int n_tiles, int nh,
                                                  int nkv, int hd, int tokens_per_tile, int window, float scale,
-                                                 const float* sink, float softcap, cudaStream_t stream) {
+                                                 const float* sink, float softcap, int keep, cudaStream_t stream) {
     if (n_tiles <= 0) return FWB_OK;
+    if (keep < 0 || (keep > 0 && window <= 0)) return FWB_BAD_ARGUMENT;
     if (!(softcap >= 0.0f)) return FWB_BAD_ARGUMENT;
     if (softcap > 0.0f && scale == 0.0f) return FWB_UNSUPPORTED;
     if (!q || !k_pool || !v_pool || !positions || !seg_start || !tile_seg || !tile_tok0 || !block_table || !out)
@@ -553,6 +557,7 @@ FWB_API int fwb_attention_prefill_tcgen05_capped(const void* q, const void* k_po
     prm.items_per_cta = (long)n_tiles * nkv <= 148 ? 1 : 2;
     prm.scale_log2 = scale * LOG2E;
     prm.sink = sink;
+    prm.keep = keep;
     prm.cap_pre = softcap > 0.0f ? scale / softcap : 0.0f;
     prm.cap_unit = softcap > 0.0f ? softcap / scale : 0.0f;
     prm.status = status_word();

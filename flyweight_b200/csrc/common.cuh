@@ -123,6 +123,22 @@ __host__ __device__ __forceinline__ int first_visible_key(int pos, int span) {
     return 0;
 }
 
+// Which key tiles (of `tile` positions) a walk from the lowest visible key `lo` to `last` touches when the
+// sequence's first `keep` positions stay visible beside a sliding window: `kept` tiles from position 0 on
+// that end before the window's first tile, then the window's own.  keep == 0: the window's alone.
+struct KeyTiles {
+    int kept, first, count;      // tile i of `count`: i while i < kept, then first + (i - kept)
+    __device__ __forceinline__ int at(int i) const { return i < kept ? i : first + (i - kept); }
+};
+__device__ __forceinline__ KeyTiles key_tiles(int lo, int last, int keep, int tile) {
+    KeyTiles w;
+    w.first = lo / tile;
+    w.kept = (keep + tile - 1) / tile;
+    if (w.kept > w.first) w.kept = w.first;
+    w.count = w.kept + last / tile + 1 - w.first;
+    return w;
+}
+
 // The tanh form of gelu: 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))).
 __device__ __forceinline__ float gelu_tanh_f32(float g) {
     return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));

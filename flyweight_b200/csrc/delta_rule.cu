@@ -266,18 +266,20 @@ delta_scan_kernel(const float* __restrict__ r, const float* __restrict__ p, floa
 template <typename TO>
 __global__ void __launch_bounds__(128)
 gated_head_norm_kernel(const float* __restrict__ o, const float* __restrict__ gate, long long gate_stride,
-                       const float* __restrict__ weight, float eps, TO* __restrict__ out, int rows, int H, int e) {
+                       const float* __restrict__ weight, float scale, float eps, TO* __restrict__ out, long long out_stride,
+                       int rows, int H, int e) {
     fwb::pdl_entry();
     const int row = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
     if (row >= rows) return;
     const int t = row / H, h = row - t * H;
     const float* src = o + (size_t)row * e;
     const float* g = gate + (size_t)t * gate_stride + (size_t)h * e;
+    TO* dst = out + (size_t)t * out_stride + (size_t)h * e;
     float ss = 0.0f;
     for (int i = lane; i < e; i += 32) ss = fmaf(src[i], src[i], ss);
     const float inv = rsqrtf(warp_sum(ss) / (float)e + eps);
     for (int i = lane; i < e; i += 32)
-        out[(size_t)row * e + i] = from_f32<TO>(((src[i] * inv) * weight[i]) * silu_f32(g[i]));
+        dst[i] = from_f32<TO>(((src[i] * inv) * (weight ? weight[i] : scale)) * silu_f32(g[i]));
 }
 
 }  // namespace
@@ -324,19 +326,23 @@ FWB_API int fwb_delta_rule(const float* p, const float* taps, const float* a_log
     return fwb_launch_status();
 }
 
-// o: [T][H][e] fp32; gate: row t at gate + t * gate_stride, [H][e] fp32; weight: [e]; out: [T][H e].
+// o: [T][H][e] fp32; gate: row t at gate + t * gate_stride, [H][e] fp32; weight: [e], or null: every channel
+// counts `scale`; out: row t at out + t * out_stride (0: H e), [H][e].
 FWB_API int fwb_gated_head_norm(const float* o, const float* gate, long long gate_stride, const float* weight,
-                                float eps, void* out, int out_bf16, int T, int H, int e, cudaStream_t stream) {
+                                float scale, float eps, void* out, int out_bf16, long long out_stride, int T, int H,
+                                int e, cudaStream_t stream) {
     if (T <= 0) return FWB_OK;
-    if (!o || !gate || !weight || !out || H <= 0 || e <= 0) return FWB_BAD_ARGUMENT;
+    if (!o || !gate || !out || H <= 0 || e <= 0) return FWB_BAD_ARGUMENT;
+    if (out_stride == 0) out_stride = (long long)H * e;
+    if (out_stride < (long long)H * e) return FWB_BAD_ARGUMENT;
     const long long rows = (long long)T * H;
     if (rows > 2147483647LL / 4) return FWB_TOO_LARGE;
     const int blocks = (int)((rows + 3) / 4);
     if (out_bf16)
-        fwb::pdl(gated_head_norm_kernel<__nv_bfloat16>, blocks, 128, 0, stream)(o, gate, gate_stride, weight, eps,
-                                                                                 (__nv_bfloat16*)out, (int)rows, H, e);
+        fwb::pdl(gated_head_norm_kernel<__nv_bfloat16>, blocks, 128, 0, stream)(
+            o, gate, gate_stride, weight, scale, eps, (__nv_bfloat16*)out, out_stride, (int)rows, H, e);
     else
-        fwb::pdl(gated_head_norm_kernel<float>, blocks, 128, 0, stream)(o, gate, gate_stride, weight, eps,
-                                                                        (float*)out, (int)rows, H, e);
+        fwb::pdl(gated_head_norm_kernel<float>, blocks, 128, 0, stream)(
+            o, gate, gate_stride, weight, scale, eps, (float*)out, out_stride, (int)rows, H, e);
     return fwb_launch_status();
 }

@@ -4,7 +4,7 @@
 //   S_t = decay_h S_(t-1) + k_t v_t^T;     o_t = S_t^T q_t
 //
 // q, k (heads x dim) and v (heads x vdim) are columns of one fp32 projection row per token; with
-// `act_silu` they pass silu on the way in.  One block owns 32 columns of one head's state for one
+// `act_silu` they pass silu on the way in, and k is multiplied by `k_scale`.  One block owns 32 columns of one head's state for one
 // segment of the step and walks the segment's tokens in order; the state's rows are cut over the
 // block's warps, 16 rows a thread, in registers.  Tokens are staged 16 at a time in shared memory, so the
 // walk itself reads no global memory; the partial read-outs of the warps are summed in warp order when
@@ -22,7 +22,7 @@ constexpr int STAGE = 16;     // tokens staged at a time
 constexpr int MAX_SPLITS = 32;
 
 __global__ void __launch_bounds__(COLS * MAX_SPLITS)
-decay_scan_kernel(const float* __restrict__ p, long long row_stride, int q_col, int k_col, int v_col, int act_silu,
+decay_scan_kernel(const float* __restrict__ p, long long row_stride, int q_col, int k_col, int v_col, int act_silu, float k_scale,
                   const float* __restrict__ decay, float* __restrict__ state, long long slot_stride,
                   const int* __restrict__ seg_start, const int* __restrict__ seg_slot, float* __restrict__ o,
                   int H, int d, int e) {
@@ -61,6 +61,7 @@ decay_scan_kernel(const float* __restrict__ p, long long row_stride, int q_col, 
                     qv = silu_f32(qv);
                     kv = silu_f32(kv);
                 }
+                kv *= k_scale;
             }
             qs[i] = qv;
             ks[i] = kv;
@@ -185,7 +186,7 @@ __device__ __forceinline__ uint2 pack4(float4 v) {
 // state's update rides on the values: S' = g^n S + sum_j k_j (g^(n-1-j) v_j)^T, so the keys enter exactly.
 template <bool SUMS, bool VEC>
 __global__ void __launch_bounds__(THREADS, 2)
-decay_runs_kernel(const float* __restrict__ p, long long row_stride, int q_col, int k_col, int v_col, int act_silu,
+decay_runs_kernel(const float* __restrict__ p, long long row_stride, int q_col, int k_col, int v_col, int act_silu, float k_scale,
                   const float* __restrict__ decay, float* __restrict__ state, long long slot_stride,
                   const int* __restrict__ seg_start, const int* __restrict__ seg_slot,
                   const int* __restrict__ piece_seg, const int* __restrict__ piece_tok0, int piece_len,
@@ -244,7 +245,9 @@ decay_runs_kernel(const float* __restrict__ p, long long row_stride, int q_col, 
                 const int i = base + u * THREADS, tok = i / d4, r = (i - tok * d4) << 2;
                 if (i >= RUN * d4) break;
                 if (!SUMS) *reinterpret_cast<uint2*>(Qs + tok * QS + r) = pack4(act_silu ? silu4(qv[u]) : qv[u]);
-                *reinterpret_cast<uint2*>(Ks + tok * QS + r) = pack4(act_silu ? silu4(kv[u]) : kv[u]);
+                const float4 key = act_silu ? silu4(kv[u]) : kv[u];
+                *reinterpret_cast<uint2*>(Ks + tok * QS + r) =
+                    pack4(make_float4(key.x * k_scale, key.y * k_scale, key.z * k_scale, key.w * k_scale));
             }
         }
         {   // v: the rounded value, and the rounded value times g^(n-1-token) in two halves
@@ -433,7 +436,7 @@ size_t decay_runs_smem(int DP) {
 // k_col and v [H][e] from v_col.  decay: fp32 [H].  state: fp32, a request's slot `slot_stride` entries after
 // the one before, [H][d][e] at its head (read at the head of every segment and advanced).  seg_start [S+1],
 // seg_slot [S]: the step's segments.  o: fp32 [T][H][e].
-FWB_API int fwb_decay_scan(const float* p, long long row_stride, int q_col, int k_col, int v_col, int act_silu,
+FWB_API int fwb_decay_scan(const float* p, long long row_stride, int q_col, int k_col, int v_col, int act_silu, float k_scale,
                            const float* decay, float* state, long long slot_stride, const int* seg_start,
                            const int* seg_slot, float* o, int T, int S, int H, int d, int e, cudaStream_t stream) {
     if (T <= 0 || S <= 0) return FWB_OK;
@@ -450,7 +453,7 @@ FWB_API int fwb_decay_scan(const float* p, long long row_stride, int q_col, int 
         if (err != cudaSuccess) return (int)err;
     }
     fwb::pdl(decay_scan_kernel, dim3(S, H, tiles), COLS * splits, smem, stream)(
-        p, row_stride, q_col, k_col, v_col, act_silu, decay, state, slot_stride, seg_start, seg_slot, o, H, d, e);
+        p, row_stride, q_col, k_col, v_col, act_silu, k_scale, decay, state, slot_stride, seg_start, seg_slot, o, H, d, e);
     return fwb_launch_status();
 }
 
@@ -459,7 +462,7 @@ FWB_API int fwb_decay_scan(const float* p, long long row_stride, int q_col, int 
 // to 256 channels (FWB_UNSUPPORTED beyond: the token-by-token form takes those).  The segments come cut into
 // `P` pieces of at most `piece_len` tokens (a multiple of 64): piece_seg, piece_tok0.  `scratch`: fp32
 // [P][H d e], needed when some segment has more than one piece (`chained` != 0), else it may be null.
-FWB_API int fwb_decay_runs(const float* p, long long row_stride, int q_col, int k_col, int v_col, int act_silu,
+FWB_API int fwb_decay_runs(const float* p, long long row_stride, int q_col, int k_col, int v_col, int act_silu, float k_scale,
                            const float* decay, float* state, long long slot_stride, const int* seg_start,
                            const int* seg_slot, const int* piece_seg, const int* piece_tok0, int piece_len,
                            int chained, float* scratch, float* o, int T, int S, int P, int H, int d, int e,
@@ -487,7 +490,7 @@ FWB_API int fwb_decay_runs(const float* p, long long row_stride, int q_col, int 
     }
     if (chained) {
         fwb::pdl(sums, dim3(P, H, tiles), THREADS, smem, stream)(
-            p, row_stride, q_col, k_col, v_col, act_silu, decay, state, slot_stride, seg_start, seg_slot, piece_seg,
+            p, row_stride, q_col, k_col, v_col, act_silu, k_scale, decay, state, slot_stride, seg_start, seg_slot, piece_seg,
             piece_tok0, piece_len, scratch, o, H, d, e, DP);
         int status = fwb_launch_status();
         if (status != FWB_OK) return status;
@@ -497,7 +500,7 @@ FWB_API int fwb_decay_runs(const float* p, long long row_stride, int q_col, int 
         if (status != FWB_OK) return status;
     }
     fwb::pdl(walk, dim3(P, H, tiles), THREADS, smem, stream)(
-        p, row_stride, q_col, k_col, v_col, act_silu, decay, state, slot_stride, seg_start, seg_slot, piece_seg,
+        p, row_stride, q_col, k_col, v_col, act_silu, k_scale, decay, state, slot_stride, seg_start, seg_slot, piece_seg,
         piece_tok0, piece_len, chained ? scratch : nullptr, o, H, d, e, DP);
     return fwb_launch_status();
 }

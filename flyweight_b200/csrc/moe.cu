@@ -6,6 +6,7 @@
 //            is its largest choice value, only the `keep` best runs stay in the race (the others count
 //            as minus infinity), and the `top` largest survivors are chosen.  The weights are the plain
 //            s of the chosen, not renormalised.  Ties go to the lower index.
+//            Optionally s = sigmoid(router h) instead, each output on its own, and no correction.
 //   sort     pairs whose output is a real expert (index < E) are counted per expert, the counts are
 //            scanned, every pair gets its row among its expert's rows, and the row tiles of the two
 //            products are listed.  Outputs from E on are identity experts: they have no row.
@@ -14,7 +15,8 @@
 //            the stacked matrix [gate rows | up rows]; form 0: the plain product in fp32.
 //   gather   the sorted rows' inputs side by side, for the grouped tensor-core product (bfloat16)
 //   combine  out[t] = sum over the token's pairs, in slot order, of weight * (expert row | h[t] itself
-//            for an identity expert); alone, or followed in the same kernel by a weighted RMS norm of
+//            for an identity expert); with weights that belong on the experts' inputs the rows were
+//            weighted on their way in (gather, or form 1 of gemm) and enter the sum as they are; alone, or followed in the same kernel by a weighted RMS norm of
 //            the sum and the residual sum, x[t] += w * unit(out[t]).
 // A pair's row is a sum over k in a fixed order whatever else is in the step, and a token's pairs are
 // added in slot order, so a token's result does not depend on the batch.  Grids are sized for the
@@ -27,12 +29,13 @@ using namespace fwb;
 namespace {
 
 constexpr int TM = 64, TN = 64, TK = 16;       // tile of the experts' products
+constexpr int SCORE_SIGMOID = 1;               // a router's scores: 0 softmax over the outputs, 1 sigmoid of each
 
 template <typename TH>
 __global__ void __launch_bounds__(512)
 moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, const float* __restrict__ correction,
                  int* __restrict__ ids, float* __restrict__ weights, int T, int W, int N, int n_groups, int keep,
-                 int top, int vec) {
+                 int top, int vec, int scoring) {
     fwb::pdl_entry();
     // One block per token.  Its warps share the router's outputs between them (output n: lanes stride
     // over k with sixteen sums in flight, added in one fixed order); warp 0 then chooses.
@@ -122,17 +125,21 @@ moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, con
     }
     __syncthreads();
     if (warp != 0) return;
-    float m = -INFINITY;
-    for (int n = lane; n < N; n += 32) m = fmaxf(m, s[n]);
-    m = warp_max(m);
-    float sum = 0.0f;
-    for (int n = lane; n < N; n += 32) sum += expf(s[n] - m);
-    sum = warp_sum(sum);
-    for (int n = lane; n < N; n += 32) {
-        const float v = expf(s[n] - m) / sum;
-        s[n] = v;
-        choice[n] = v + correction[n];
+    if (scoring == SCORE_SIGMOID) {
+        for (int n = lane; n < N; n += 32) {
+            const float z = s[n], e = expf(-fabsf(z));
+            s[n] = z >= 0.0f ? 1.0f / (1.0f + e) : e / (1.0f + e);
+        }
+    } else {
+        float m = -INFINITY;
+        for (int n = lane; n < N; n += 32) m = fmaxf(m, s[n]);
+        m = warp_max(m);
+        float sum = 0.0f;
+        for (int n = lane; n < N; n += 32) sum += expf(s[n] - m);
+        sum = warp_sum(sum);
+        for (int n = lane; n < N; n += 32) s[n] = expf(s[n] - m) / sum;
     }
+    for (int n = lane; n < N; n += 32) choice[n] = s[n] + (correction ? correction[n] : 0.0f);
     __syncwarp();
     const int per = N / n_groups;
     for (int g = lane; g < n_groups; g += 32) {
@@ -213,9 +220,11 @@ moe_route_table_kernel(const int* __restrict__ token_ids, const int* __restrict_
 //   pair_row[A]      sorted row of every pair (-1: an identity expert)
 //   tiles[0]         number of row tiles (of tile_rows rows at most, none across two experts);
 //                    tiles[1 + 2 i], tiles[2 + 2 i]: expert and first row of tile i
+//   row_weight[A]    the pair's weight at its sorted row (only with `row_weight`)
 __global__ void __launch_bounds__(1024)
 moe_sort_kernel(const int* __restrict__ ids, int A, int top, int E, int tile_rows, int* __restrict__ offsets,
-                int* __restrict__ row_token, int* __restrict__ pair_row, int* __restrict__ tiles) {
+                int* __restrict__ row_token, int* __restrict__ pair_row, int* __restrict__ tiles,
+                const float* __restrict__ weights, float* __restrict__ row_weight) {
     fwb::pdl_entry();
     extern __shared__ int counts[];               // [E] counts, then [E] cursors
     int* cursor = counts + E;
@@ -249,6 +258,7 @@ moe_sort_kernel(const int* __restrict__ ids, int A, int top, int E, int tile_row
         if (e >= 0 && e < E) {
             row = atomicAdd(&cursor[e], 1);
             row_token[row] = a / top;
+            if (row_weight) row_weight[row] = weights[a];
         }
         pair_row[a] = row;
     }
@@ -256,12 +266,26 @@ moe_sort_kernel(const int* __restrict__ ids, int A, int top, int E, int tile_row
 
 __global__ void __launch_bounds__(128)
 moe_gather_rows_kernel(const uint4* __restrict__ h, const int* __restrict__ row_token, const int* __restrict__ offsets,
-                       int E, uint4* __restrict__ out, int pieces) {
+                       int E, uint4* __restrict__ out, int pieces, const float* __restrict__ row_weight) {
     fwb::pdl_entry();
     const int row = blockIdx.x;
     if (row >= offsets[E]) return;            // rows behind the last expert's belong to nobody
     const uint4* src = h + (size_t)row_token[row] * pieces;
-    for (int i = threadIdx.x; i < pieces; i += blockDim.x) out[(size_t)row * pieces + i] = src[i];
+    if (!row_weight) {
+        for (int i = threadIdx.x; i < pieces; i += blockDim.x) out[(size_t)row * pieces + i] = src[i];
+        return;
+    }
+    const float w = row_weight[row];
+    for (int i = threadIdx.x; i < pieces; i += blockDim.x) {
+        uint4 bits = src[i];
+        __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&bits);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float2 v = __bfloat1622float2(h2[j]);
+            h2[j] = __floats2bfloat162_rn(v.x * w, v.y * w);
+        }
+        out[(size_t)row * pieces + i] = bits;
+    }
 }
 
 // FORM 1: out[row][f] = act(x . gate_f) * (x . up_f), w: [E][2F][K] (gate rows, then up rows), N = F.
@@ -271,7 +295,7 @@ template <typename TX, typename TW, typename TO, int FORM>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TO* __restrict__ out,
                 const int* __restrict__ offsets, const int* __restrict__ row_token, const int* __restrict__ tiles,
-                int N, int K, int act, float limit) {
+                int N, int K, int act, float limit, const float* __restrict__ row_weight) {
     fwb::pdl_entry();
     const int tile = blockIdx.y;
     if (tile >= tiles[0]) return;
@@ -281,8 +305,10 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TO* __restri
     __shared__ float xs[TK][TM + 1];
     __shared__ float ws[FORM ? 2 : 1][TK][TN + 1];
     __shared__ int src_row[TM];
+    __shared__ float src_weight[TM];              // what the row's input is multiplied by (FORM 1)
     if (threadIdx.x < TM) {
         const int row = row0 + threadIdx.x;
+        src_weight[threadIdx.x] = (FORM && row_weight && row < row_end) ? row_weight[row] : 1.0f;
         src_row[threadIdx.x] = row < row_end ? (FORM ? row_token[row] : row) : -1;
     }
     __syncthreads();
@@ -294,7 +320,8 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TO* __restri
         for (int i = threadIdx.x; i < TM * TK; i += 256) {
             const int r = i / TK, k = i - r * TK;
             const int src = src_row[r];
-            xs[k][r] = (src >= 0 && k0 + k < K) ? to_f32<TX>(x[(size_t)src * K + k0 + k]) : 0.0f;
+            const float v = (src >= 0 && k0 + k < K) ? to_f32<TX>(x[(size_t)src * K + k0 + k]) : 0.0f;
+            xs[k][r] = FORM ? v * src_weight[r] : v;
         }
         for (int i = threadIdx.x; i < TN * TK; i += 256) {
             const int n = i / TK, k = i - n * TK;
@@ -342,7 +369,7 @@ template <typename TH>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, const TH* __restrict__ h, const int* __restrict__ pair_row,
                    const int* __restrict__ ids, const float* __restrict__ weights, float* __restrict__ out, int W,
-                   int top, int E) {
+                   int top, int E, int weighted_in) {
     fwb::pdl_entry();
     constexpr int MAX_TOP = 64;
     __shared__ int rows[MAX_TOP];                 // the sorted row of every slot; -1: identity; -2: nothing
@@ -352,7 +379,7 @@ moe_combine_kernel(const float* __restrict__ y, const TH* __restrict__ h, const 
         const int a = t * top + threadIdx.x;
         const int row = pair_row[a];
         rows[threadIdx.x] = row >= 0 ? row : (ids[a] >= E ? -1 : -2);
-        wts[threadIdx.x] = weights[a];
+        wts[threadIdx.x] = weighted_in && row >= 0 ? 1.0f : weights[a];
     }
     __syncthreads();
     if ((W & 3) == 0 && sizeof(TH) == 4) {
@@ -425,7 +452,7 @@ __global__ void __launch_bounds__(256)
 moe_combine_norm_add_kernel(const float* __restrict__ y, const TH* __restrict__ h, const int* __restrict__ pair_row,
                             const int* __restrict__ ids, const float* __restrict__ weights, float* __restrict__ x,
                             const float* __restrict__ norm_w, float eps, int W, int top, int E,
-                            const float* __restrict__ extra) {
+                            const float* __restrict__ extra, int weighted_in) {
     fwb::pdl_entry();
     constexpr int MAX_TOP = 64;
     extern __shared__ float sum_row[];            // [W]
@@ -437,7 +464,7 @@ moe_combine_norm_add_kernel(const float* __restrict__ y, const TH* __restrict__ 
         const int a = t * top + threadIdx.x;
         const int row = pair_row[a];
         rows[threadIdx.x] = row >= 0 ? row : (ids[a] >= E ? -1 : -2);
-        wts[threadIdx.x] = weights[a];
+        wts[threadIdx.x] = weighted_in && row >= 0 ? 1.0f : weights[a];
     }
     __syncthreads();
     float ss = 0.0f;
@@ -482,12 +509,13 @@ moe_combine_norm_add_kernel(const float* __restrict__ y, const TH* __restrict__ 
 
 }  // namespace
 
-// h: [T][W] fp32 or bf16; router: [N][W] fp32; correction: [N] fp32; ids, weights: [T][top].
+// h: [T][W] fp32 or bf16; router: [N][W] fp32; correction: [N] fp32 or null; ids, weights: [T][top].
+// scoring: 0 softmax over the outputs, 1 the sigmoid of each.
 FWB_API int fwb_moe_route(const void* h, int h_bf16, const float* router, const float* correction, int* ids,
-                          float* weights, int T, int W, int N, int n_groups, int keep, int top,
+                          float* weights, int T, int W, int N, int n_groups, int keep, int top, int scoring,
                           cudaStream_t stream) {
     if (T <= 0) return FWB_OK;
-    if (!h || !router || !correction || !ids || !weights) return FWB_BAD_ARGUMENT;
+    if (!h || !router || !ids || !weights || scoring < 0 || scoring > 1) return FWB_BAD_ARGUMENT;
     if (W <= 0 || N <= 0 || n_groups <= 0 || N % n_groups || keep <= 0 || keep > n_groups || top <= 0 ||
         top > keep * (N / n_groups))
         return FWB_BAD_ARGUMENT;
@@ -502,10 +530,10 @@ FWB_API int fwb_moe_route(const void* h, int h_bf16, const float* router, const 
     if (smem > 48 * 1024) return FWB_TOO_LARGE;
     if (h_bf16)
         fwb::pdl(moe_route_kernel<__nv_bfloat16>, blocks, threads, smem, stream)(
-            (const __nv_bfloat16*)h, router, correction, ids, weights, T, W, N, n_groups, keep, top, vec);
+            (const __nv_bfloat16*)h, router, correction, ids, weights, T, W, N, n_groups, keep, top, vec, scoring);
     else
         fwb::pdl(moe_route_kernel<float>, blocks, threads, smem, stream)((const float*)h, router, correction, ids,
-                                                                          weights, T, W, N, n_groups, keep, top, vec);
+                                                                          weights, T, W, N, n_groups, keep, top, vec, scoring);
     return fwb_launch_status();
 }
 
@@ -520,33 +548,38 @@ FWB_API int fwb_moe_route_table(const int* token_ids, const int* table, int voca
 
 // ids: [A]; offsets: [E + 1]; row_token, pair_row: [A]; tiles: [1 + 2 (A / tile_rows + E + 1)].
 // tile_rows: rows of a tile of the products that follow (TM = 64 for fwb_moe_gemm).
+// weights [A], row_weight [A]: both or neither; row_weight receives every sorted row's pair weight.
 FWB_API int fwb_moe_sort(const int* ids, int A, int top, int E, int tile_rows, int* offsets, int* row_token,
-                         int* pair_row, int* tiles, cudaStream_t stream) {
+                         int* pair_row, int* tiles, const float* weights, float* row_weight, cudaStream_t stream) {
     if (A <= 0) return FWB_OK;
-    if (!ids || !offsets || !row_token || !pair_row || !tiles || top <= 0 || E < 0 || tile_rows <= 0)
+    if (!ids || !offsets || !row_token || !pair_row || !tiles || top <= 0 || E < 0 || tile_rows <= 0 ||
+        (weights == nullptr) != (row_weight == nullptr))
         return FWB_BAD_ARGUMENT;
     if (E > 4096) return FWB_TOO_LARGE;
     fwb::pdl(moe_sort_kernel, 1, 1024, (size_t)(2 * E + 1) * sizeof(int), stream)(ids, A, top, E, tile_rows, offsets,
-                                                                                  row_token, pair_row, tiles);
+                                                                                  row_token, pair_row, tiles, weights,
+                                                                                  row_weight);
     return fwb_launch_status();
 }
 
 // out[row] = h[row_token[row]] for the sorted rows (16-byte pieces): the experts' first product then
-// reads its rows side by side.  h: [T][W] bf16, W a multiple of 8; out: [A][W].
+// reads its rows side by side.  h: [T][W] bf16, W a multiple of 8; out: [A][W].  row_weight: [A] or null;
+// row i is multiplied by row_weight[i] and rounded once more.
 FWB_API int fwb_moe_gather_rows(const void* h, const int* row_token, const int* offsets, int E, void* out, int A,
-                                int W, cudaStream_t stream) {
+                                int W, const float* row_weight, cudaStream_t stream) {
     if (A <= 0) return FWB_OK;
     if (!h || !row_token || !offsets || !out || W <= 0 || (W & 7)) return FWB_BAD_ARGUMENT;
-    fwb::pdl(moe_gather_rows_kernel, A, 128, 0, stream)((const uint4*)h, row_token, offsets, E, (uint4*)out, W / 8);
+    fwb::pdl(moe_gather_rows_kernel, A, 128, 0, stream)((const uint4*)h, row_token, offsets, E, (uint4*)out, W / 8,
+                                                         row_weight);
     return fwb_launch_status();
 }
 
 // form 1: x [T][K] (rows gathered by row_token), w [E][2N][K], out [A][N] in the dtype of x.
 // form 0: x [A][K] sorted rows, w [E][N][K], out [A][N] fp32.
-// x and w are both fp32 or both bf16.  max_tiles: the most tiles the sorted list can hold (the grid).
+// x and w are both fp32 or both bf16.  row_weight: [A] or null, multiplies the inputs of form 1.  max_tiles: the most tiles the sorted list can hold (the grid).
 FWB_API int fwb_moe_gemm(const void* x, const void* w, int bf16, void* out, const int* offsets,
                          const int* row_token, const int* tiles, int max_tiles, int N, int K, int form, int act,
-                         float limit, cudaStream_t stream) {
+                         float limit, const float* row_weight, cudaStream_t stream) {
     if (max_tiles <= 0) return FWB_OK;
     if (!x || !w || !out || !offsets || !row_token || !tiles || N <= 0 || K <= 0 || form < 0 || form > 1 ||
         act < 0 || act > 2)
@@ -556,31 +589,32 @@ FWB_API int fwb_moe_gemm(const void* x, const void* w, int bf16, void* out, cons
     using bf = __nv_bfloat16;
     if (form == 1 && bf16)
         fwb::pdl(moe_gemm_kernel<bf, bf, bf, 1>, grid, 256, 0, stream)((const bf*)x, (const bf*)w, (bf*)out, offsets,
-                                                                       row_token, tiles, N, K, act, limit);
+                                                                       row_token, tiles, N, K, act, limit, row_weight);
     else if (form == 1)
         fwb::pdl(moe_gemm_kernel<float, float, float, 1>, grid, 256, 0, stream)(
-            (const float*)x, (const float*)w, (float*)out, offsets, row_token, tiles, N, K, act, limit);
+            (const float*)x, (const float*)w, (float*)out, offsets, row_token, tiles, N, K, act, limit, row_weight);
     else if (bf16)
         fwb::pdl(moe_gemm_kernel<bf, bf, float, 0>, grid, 256, 0, stream)((const bf*)x, (const bf*)w, (float*)out,
-                                                                          offsets, row_token, tiles, N, K, act, limit);
+                                                                          offsets, row_token, tiles, N, K, act, limit, row_weight);
     else
         fwb::pdl(moe_gemm_kernel<float, float, float, 0>, grid, 256, 0, stream)(
-            (const float*)x, (const float*)w, (float*)out, offsets, row_token, tiles, N, K, act, limit);
+            (const float*)x, (const float*)w, (float*)out, offsets, row_token, tiles, N, K, act, limit, row_weight);
     return fwb_launch_status();
 }
 
-// y: [A][W] fp32 sorted rows; h: [T][W]; out: [T][W] fp32.
+// y: [A][W] fp32 sorted rows; h: [T][W]; out: [T][W] fp32.  weighted_in: the rows were weighted on their way in.
 FWB_API int fwb_moe_combine(const float* y, const void* h, int h_bf16, const int* pair_row, const int* ids,
-                            const float* weights, float* out, int T, int W, int top, int E, cudaStream_t stream) {
+                            const float* weights, float* out, int T, int W, int top, int E, int weighted_in,
+                            cudaStream_t stream) {
     if (T <= 0) return FWB_OK;
     if (!y || !h || !pair_row || !ids || !weights || !out || W <= 0 || top <= 0) return FWB_BAD_ARGUMENT;
     if (top > 64) return FWB_TOO_LARGE;
     if (h_bf16)
         fwb::pdl(moe_combine_kernel<__nv_bfloat16>, T, 256, 0, stream)(y, (const __nv_bfloat16*)h, pair_row, ids,
-                                                                       weights, out, W, top, E);
+                                                                       weights, out, W, top, E, weighted_in);
     else
         fwb::pdl(moe_combine_kernel<float>, T, 256, 0, stream)(y, (const float*)h, pair_row, ids, weights, out, W,
-                                                               top, E);
+                                                               top, E, weighted_in);
     return fwb_launch_status();
 }
 
@@ -588,7 +622,7 @@ FWB_API int fwb_moe_combine(const float* y, const void* h, int h_bf16, const int
 // x[t] += norm_w * sum / sqrt(mean(sum^2) + eps) in place (x: [T][W] fp32).
 FWB_API int fwb_moe_combine_norm_add(const float* y, const void* h, int h_bf16, const int* pair_row, const int* ids,
                                      const float* weights, float* x, const float* norm_w, float eps, int T, int W,
-                                     int top, int E, const float* extra, cudaStream_t stream) {
+                                     int top, int E, const float* extra, int weighted_in, cudaStream_t stream) {
     if (T <= 0) return FWB_OK;
     if (!y || !h || !pair_row || !ids || !weights || !x || !norm_w || W <= 0 || top <= 0) return FWB_BAD_ARGUMENT;
     if (top > 64) return FWB_TOO_LARGE;
@@ -598,12 +632,12 @@ FWB_API int fwb_moe_combine_norm_add(const float* y, const void* h, int h_bf16, 
         if (smem > 48 * 1024)
             cudaFuncSetAttribute(moe_combine_norm_add_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         fwb::pdl(moe_combine_norm_add_kernel<__nv_bfloat16>, T, 256, smem, stream)(
-            y, (const __nv_bfloat16*)h, pair_row, ids, weights, x, norm_w, eps, W, top, E, extra);
+            y, (const __nv_bfloat16*)h, pair_row, ids, weights, x, norm_w, eps, W, top, E, extra, weighted_in);
     } else {
         if (smem > 48 * 1024)
             cudaFuncSetAttribute(moe_combine_norm_add_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         fwb::pdl(moe_combine_norm_add_kernel<float>, T, 256, smem, stream)(y, (const float*)h, pair_row, ids, weights, x,
-                                                                           norm_w, eps, W, top, E, extra);
+                                                                           norm_w, eps, W, top, E, extra, weighted_in);
     }
     return fwb_launch_status();
 }

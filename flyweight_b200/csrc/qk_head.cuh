@@ -99,4 +99,37 @@ __device__ __forceinline__ void head_norm_rope8(float (&v)[8], bool valid, int k
     }
 }
 
+// A plain rotation of a head's first `rot` channels (no norm), for rotated values: the same lanes own the
+// same channels as above, every lane of the warp must call this, lanes whose head does not turn (`on`
+// false) keep what they hold.  Needs rot % 16 == 0.
+__device__ __forceinline__ void head_turn8(float (&v)[8], bool on, int gl, int rot, int pairing,
+                                           const float2* __restrict__ cs) {
+    const int lane = threadIdx.x & 31;
+    const int half_lanes = rot >> 4, rot_lanes = rot >> 3;
+    if (pairing) {
+        if (!on || gl >= rot_lanes) return;
+        const float2* c = cs + gl * 4;
+#pragma unroll
+        for (int j = 0; j < 4; ++j) {
+            const float2 a = c[j];
+            const float x0 = v[2 * j], x1 = v[2 * j + 1];
+            v[2 * j] = x0 * a.x - x1 * a.y;
+            v[2 * j + 1] = x1 * a.x + x0 * a.y;
+        }
+        return;
+    }
+    const int partner = gl < half_lanes ? lane + half_lanes : (gl < rot_lanes ? lane - half_lanes : lane);
+    float other[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) other[i] = __shfl_sync(0xffffffffu, v[i], partner & 31);
+    if (!on || gl >= rot_lanes) return;
+    const bool low = gl < half_lanes;
+    const float2* c = cs + (low ? gl : gl - half_lanes) * 8;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const float2 a = c[i];
+        v[i] = low ? v[i] * a.x - other[i] * a.y : v[i] * a.x + other[i] * a.y;
+    }
+}
+
 }  // namespace fwb

@@ -70,6 +70,14 @@ def force_tiled(flag: bool) -> None:
     lib.set_option("force_tiled", _force_tiled)
 
 
+def window_tiles(max_tiles: int, window: int, keep_first: int = 0) -> int:
+    """How many 64-key tiles a decoded token walks at most: the block table's width, or with a sliding
+    window the tiles it can touch (and those of the kept first positions)."""
+    if window <= 0:
+        return max_tiles
+    return min(max_tiles, (window + 62) // 64 + 1 + -(-keep_first // 64))
+
+
 def decode_splits(n_tokens: int, n_kv: int, max_tiles: int, head_dim: int = 64):
     """How many slices of the context run as separate CTAs: (slices, tiles per slice, merged inside the
     kernel by a cluster).  Depends only on static sizes of the step (tokens, KV heads, block-table
@@ -172,13 +180,15 @@ def tensor_core_shape_ok(n_heads: int, n_kv: int, head_dim: int, page_size: int)
     return groups is not None and ops.attention_mma_shape_ok(n_heads, groups, head_dim, page_size)
 
 
-def paged_attention(ctx, q, cache, block_table, n_heads, window, scale, out_dtype, sink=None, softcap=0.0):
+def paged_attention(ctx, q, cache, block_table, n_heads, window, scale, out_dtype, sink=None, softcap=0.0,
+                    keep_first=0):
     """Causal GQA of every token of the step over its request's pages.  ``window`` is the kernels' one
     mask parameter: > 0 a sliding window of that many positions, < 0 chunks of ``-window`` positions
     counted from position 0 (a query sees its own chunk up to itself), 0 every earlier key.  A cache with one pool
     (``v_pool`` None) holds rows that serve as keys and as values.  ``sink``: fp32 [n_heads], a score
     per head that joins every softmax denominator (not scaled, no value).  ``softcap`` > 0: scores become
-    ``softcap * tanh(score / softcap)`` behind the scale (the sink is not capped)."""
+    ``softcap * tanh(score / softcap)`` behind the scale (the sink is not capped).  ``keep_first`` > 0
+    (with a sliding window): the sequence's first that many positions stay visible to every query."""
     batch = ctx.batch
     k_pool = cache.k_pool
     v_pool = cache.v_pool if cache.v_pool is not None else k_pool
@@ -188,12 +198,17 @@ def paged_attention(ctx, q, cache, block_table, n_heads, window, scale, out_dtyp
     if sink is not None or n_kv != pool_heads:
         extra = {"sink": sink, "groups": n_kv}
     capped = {"softcap": float(softcap)} if softcap else {}
+    if keep_first:
+        if window <= 0:
+            raise ops.KernelError("kept first positions go with a sliding window")
+        capped["keep_first"] = int(keep_first)
     extra.update(capped)
+    walked = window_tiles(block_table.shape[1], window, keep_first)
     if (_use_mma and q.dtype == torch.bfloat16 and k_pool.dtype == torch.bfloat16
             and out_dtype == torch.bfloat16
             and ops.attention_mma_shape_ok(n_heads, n_kv, head_dim, page_size)):
         if batch.max_segment == 1 and not _force_tiled:
-            splits, tiles_per_split, in_cluster = decode_splits(batch.n_tokens, n_kv, block_table.shape[1], head_dim)
+            splits, tiles_per_split, in_cluster = decode_splits(batch.n_tokens, n_kv, walked, head_dim)
             return ops.attention_decode_mma(q, k_pool, v_pool, batch.positions, batch.tok_seg,
                                             block_table, n_heads, window, scale, splits,
                                             tiles_per_split, in_cluster, **extra)
@@ -206,7 +221,7 @@ def paged_attention(ctx, q, cache, block_table, n_heads, window, scale, out_dtyp
             # portions of prompts behind them the tiled kernels; both write their rows of `out`
             first = batch.leading_singles
             out = torch.empty_like(q)
-            splits, tiles_per_split, in_cluster = decode_splits(first, n_kv, block_table.shape[1], head_dim)
+            splits, tiles_per_split, in_cluster = decode_splits(first, n_kv, walked, head_dim)
             ops.attention_decode_mma(q, k_pool, v_pool, batch.positions, batch.tok_seg, block_table,
                                      n_heads, window, scale, splits, tiles_per_split, in_cluster,
                                      out=out, n_tokens=first, **extra)
@@ -228,4 +243,5 @@ def paged_attention(ctx, q, cache, block_table, n_heads, window, scale, out_dtyp
                                          tile_seg, tile_tok0, n_tiles, tokens_per_tile, block_table,
                                          n_heads, window, scale, out=out, **extra)
     return ops.attention_simt(q, k_pool, v_pool, batch.positions, batch.tok_seg, block_table,
-                              n_heads, window, scale, out_dtype, sink=sink, softcap=softcap)
+                              n_heads, window, scale, out_dtype, sink=sink, softcap=softcap,
+                              keep_first=keep_first)

@@ -2,6 +2,8 @@
 (token, expert) pairs, the experts' products over the sorted rows, the weighted sum."""
 from __future__ import annotations
 
+from typing import Optional
+
 import torch
 
 from . import lib
@@ -19,19 +21,26 @@ def set_tensor_cores(flag: bool) -> None:
     _use_tensor_cores = bool(flag)
 
 
-def route(h: torch.Tensor, router: torch.Tensor, correction: torch.Tensor, n_groups: int, keep: int, top: int):
-    """ids int32 [T][top] and weights fp32 [T][top]: softmax scores over all router outputs; the choice
-    on score + correction inside the ``keep`` best of ``n_groups`` runs of neighbours; the weights are
-    the chosen outputs' plain scores."""
+ROUTER_SCORES = {"softmax": 0, "sigmoid": 1}
+
+
+def route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], n_groups: int, keep: int, top: int,
+          scores: str = "softmax"):
+    """ids int32 [T][top] and weights fp32 [T][top]: ``scores`` "softmax" over all router outputs or the
+    "sigmoid" of each; the choice on score (+ correction) inside the ``keep`` best of ``n_groups`` runs of
+    neighbours; the weights are the chosen outputs' plain scores."""
     check_tensor("router input", h)
     T, W = h.shape
     N = router.shape[0]
     check_tensor("router", router, torch.float32, (N, W))
-    check_tensor("router correction", correction, torch.float32, (N,))
+    if correction is not None:
+        check_tensor("router correction", correction, torch.float32, (N,))
+    if scores not in ROUTER_SCORES:
+        raise KernelError(f"unknown router scores {scores!r}; known: " + ", ".join(ROUTER_SCORES))
     ids = torch.empty((T, top), dtype=torch.int32, device=h.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=h.device)
     lib.call("fwb_moe_route", ptr(h), is_bf16(h), ptr(router), ptr(correction), ptr(ids), ptr(weights), T, W, N,
-             int(n_groups), int(keep), int(top), stream())
+             int(n_groups), int(keep), int(top), ROUTER_SCORES[scores], stream())
     return ids, weights
 
 
@@ -51,13 +60,15 @@ def route_table(token_ids: torch.Tensor, table: torch.Tensor, top: int):
 
 
 def experts_forward(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
-                    w_down: torch.Tensor, activation: str = "silu", add_normed_into=None, limit: float = 0.0):
+                    w_down: torch.Tensor, activation: str = "silu", add_normed_into=None, limit: float = 0.0,
+                    weights_on: str = "output"):
     """``sum_slot weights * expert(h)`` as fp32 [T][W].  ``w_gate_up``: [E][2F][W] (gate rows, then up
     rows), ``w_down``: [E][W][F], both in the dtype of ``h``.  Router outputs from E on are identity
     experts: they pass ``h`` itself on.  ``add_normed_into`` = (x, norm weight, eps): the sum is not
     returned but normed and added, ``x += weight * sum / sqrt(mean(sum^2) + eps)`` in fp32, by the kernel
     that makes it (returns None); a fourth entry, fp32 [T][W], is added to every token's sum first (the output of an
-    expert that every token shares)."""
+    expert that every token shares).  ``weights_on`` "input": a pair's weight multiplies what the expert reads,
+    ``sum_slot expert(weights * h)``, and the experts' rows are added as they are."""
     check_tensor("expert input", h)
     T, W = h.shape
     top = ids.shape[1]
@@ -82,14 +93,19 @@ def experts_forward(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w
     meta = torch.empty(E + 1 + 2 * A + 1 + 2 * max_tiles, dtype=torch.int32, device=dev)
     offsets, row_token = meta[:E + 1], meta[E + 1:E + 1 + A]
     pair_row, tiles = meta[E + 1 + A:E + 1 + 2 * A], meta[E + 1 + 2 * A:]
+    if weights_on not in ("output", "input"):
+        raise KernelError(f"expert weights go on the output or on the input, not on {weights_on!r}")
+    weighted_in = 1 if weights_on == "input" else 0
+    row_weight = torch.empty(A, dtype=torch.float32, device=dev) if weighted_in else None
     lib.call("fwb_moe_sort", ptr(ids), A, top, E, tile_rows, ptr(offsets), ptr(row_token), ptr(pair_row), ptr(tiles),
-             stream())
+             ptr(weights) if weighted_in else None, ptr(row_weight), stream())
     a = torch.empty((A, F), dtype=h.dtype, device=dev)
     y = torch.empty((A, W), dtype=torch.float32, device=dev)
     if tensor_cores:
         from .tensorcore import EPI_F32, _gated_epilogue
         rows = torch.empty((A, W), dtype=h.dtype, device=dev)
-        lib.call("fwb_moe_gather_rows", ptr(h), ptr(row_token), ptr(offsets), E, ptr(rows), A, W, stream())
+        lib.call("fwb_moe_gather_rows", ptr(h), ptr(row_token), ptr(offsets), E, ptr(rows), A, W, ptr(row_weight),
+                 stream())
         lib.call("fwb_gemm_tcgen05_grouped", ptr(rows), ptr(w_gate_up), ptr(a), ptr(offsets), ptr(tiles), max_tiles,
                  tile_rows, A, F, W, E, 2 * F, F, _gated_epilogue(activation), F, c_float(limit), stream(),
                  tag=f"experts gate|up {F}x{W}")
@@ -97,9 +113,9 @@ def experts_forward(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w
                  tile_rows, A, W, F, E, W, W, EPI_F32, 0, c_float(0.0), stream(), tag=f"experts down {W}x{F}")
     elif E > 0:                                 # (a router may have identity experts only)
         lib.call("fwb_moe_gemm", ptr(h), ptr(w_gate_up), bf16, ptr(a), ptr(offsets), ptr(row_token), ptr(tiles),
-                 max_tiles, F, W, 1, act, c_float(limit), stream())
+                 max_tiles, F, W, 1, act, c_float(limit), ptr(row_weight), stream())
         lib.call("fwb_moe_gemm", ptr(a), ptr(w_down), bf16, ptr(y), ptr(offsets), ptr(row_token), ptr(tiles),
-                 max_tiles, W, F, 0, 0, c_float(0.0), stream())
+                 max_tiles, W, F, 0, 0, c_float(0.0), None, stream())
     if add_normed_into is not None:
         x, norm_weight, eps = add_normed_into[:3]
         extra = add_normed_into[3] if len(add_normed_into) > 3 else None
@@ -108,9 +124,9 @@ def experts_forward(h: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w
         if extra is not None:
             check_tensor("shared output", extra, torch.float32, (T, W))
         lib.call("fwb_moe_combine_norm_add", ptr(y), ptr(h), bf16, ptr(pair_row), ptr(ids), ptr(weights), ptr(x),
-                 ptr(norm_weight), c_float(eps), T, W, top, E, ptr(extra), stream())
+                 ptr(norm_weight), c_float(eps), T, W, top, E, ptr(extra), weighted_in, stream())
         return None
     out = torch.empty((T, W), dtype=torch.float32, device=dev)
     lib.call("fwb_moe_combine", ptr(y), ptr(h), bf16, ptr(pair_row), ptr(ids), ptr(weights), ptr(out), T, W, top,
-             E, stream())
+             E, weighted_in, stream())
     return out

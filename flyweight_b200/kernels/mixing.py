@@ -1,7 +1,8 @@
 """Python faces of ``csrc/layer_mix.cu`` and ``csrc/linear_attention.cu``: the small fp32 kernels of
 layers whose sublayers run side by side (norms over column ranges of a projection, values mixed between
 layers, sigmoid gates, scaled residual sums, a token-indexed side input, the mean of two normed
-outputs) and the decayed linear-attention recurrence with its gated norm."""
+outputs), the decayed linear-attention recurrence with its gated norm (``csrc/gated_average.cu`` and
+``csrc/place_heads.cu``: the gated average over time, and head outputs placed into a shared row)."""
 from __future__ import annotations
 
 from typing import Optional
@@ -204,10 +205,10 @@ def gated_rmsnorm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps
 
 
 def decay_scan(p: torch.Tensor, q_col: int, k_col: int, v_col: int, decay: torch.Tensor, state: torch.Tensor,
-               batch, heads: int, dim: int, vdim: int, act_silu: bool = True) -> torch.Tensor:
+               batch, heads: int, dim: int, vdim: int, act_silu: bool = True, k_scale: float = 1.0) -> torch.Tensor:
     """``S <- decay_h S + k v^T; o = S^T q`` over the step's ragged segments.  ``p``: fp32 [T][...] whose
     columns from ``q_col``, ``k_col`` (heads x dim each) and ``v_col`` (heads x vdim) are the projections
-    (``act_silu``: silu on the way in); ``state``: fp32 [slots][>= heads dim vdim], read at the head of
+    (``act_silu``: silu on the way in; ``k_scale`` multiplies k); ``state``: fp32 [slots][>= heads dim vdim], read at the head of
     every segment and advanced.  Returns o, fp32 [T][heads vdim]."""
     check_tensor("projection", p, torch.float32)
     T, width = p.shape
@@ -224,7 +225,7 @@ def decay_scan(p: torch.Tensor, q_col: int, k_col: int, v_col: int, decay: torch
     _i32("seg_slot", batch.seg_slot, S)
     o = torch.empty((T, heads * vdim), dtype=torch.float32, device=p.device)
     lib.call("fwb_decay_scan", ptr(p), c_longlong(width), int(q_col), int(k_col), int(v_col), 1 if act_silu else 0,
-             ptr(decay), ptr(state), c_longlong(stride), ptr(batch.seg_start), ptr(batch.seg_slot), ptr(o), T, S,
+             c_float(k_scale), ptr(decay), ptr(state), c_longlong(stride), ptr(batch.seg_start), ptr(batch.seg_slot), ptr(o), T, S,
              heads, dim, vdim, stream())
     return o
 
@@ -233,7 +234,7 @@ PIECE_TOKENS = 256      # tokens of a segment that one block of the tensor-core 
 
 
 def decay_runs(p: torch.Tensor, q_col: int, k_col: int, v_col: int, decay: torch.Tensor, state: torch.Tensor,
-               batch, heads: int, dim: int, vdim: int, act_silu: bool = True) -> torch.Tensor:
+               batch, heads: int, dim: int, vdim: int, act_silu: bool = True, k_scale: float = 1.0) -> torch.Tensor:
     """``decay_scan`` for steps that bring portions of prompts, on tensor cores: q, k and v enter the
     products as bfloat16, the state and every sum stay fp32.  Segments longer than ``PIECE_TOKENS`` are cut
     into pieces that run side by side (their contributions to the state are chained first)."""
@@ -255,9 +256,68 @@ def decay_runs(p: torch.Tensor, q_col: int, k_col: int, v_col: int, decay: torch
     scratch = torch.empty((pieces, size), dtype=torch.float32, device=p.device) if chained else None
     o = torch.empty((T, heads * vdim), dtype=torch.float32, device=p.device)
     lib.call("fwb_decay_runs", ptr(p), c_longlong(width), int(q_col), int(k_col), int(v_col), 1 if act_silu else 0,
-             ptr(decay), ptr(state), c_longlong(stride), ptr(batch.seg_start), ptr(batch.seg_slot),
+             c_float(k_scale), ptr(decay), ptr(state), c_longlong(stride), ptr(batch.seg_start), ptr(batch.seg_slot),
              ptr(piece_seg), ptr(piece_tok0), PIECE_TOKENS, 1 if chained else 0,
              ptr(scratch) if chained else None, ptr(o), T, S, pieces, heads, dim, vdim, stream())
     if chained:
         lib.add_launches(2)
     return o
+
+
+def gated_average(p: torch.Tensor, z_col: int, x_col: int, g_col: int, z_bias: Optional[torch.Tensor],
+                  x_bias: Optional[torch.Tensor], state: torch.Tensor, batch, width: int, out_dtype: torch.dtype,
+                  out_width: int = 0) -> torch.Tensor:
+    """The minGRU recurrence over the step's ragged segments.  ``p``: fp32 rows [T][...] whose columns from
+    ``z_col``, ``x_col`` and ``g_col`` (``width`` each) are the projections; per channel z = sigmoid(p_z +
+    z_bias), u = p_x + x_bias, candidate = u + 1/2 where u >= 0 else sigmoid(u), S <- (1 - z) S + z candidate;
+    returns S * silu(p_g), [T][out_width or width] (zeros behind ``width``).  ``state``: fp32 [slots][>=
+    width], read at the head of every segment and advanced."""
+    check_tensor("projection", p, torch.float32)
+    T, columns = p.shape
+    if max(z_col, x_col, g_col) + width > columns:
+        raise KernelError("the projection's rows are shorter than the columns asked for")
+    for name, t in (("z bias", z_bias), ("x bias", x_bias)):
+        if t is not None:
+            check_tensor(name, t, torch.float32, (width,))
+    if (not state.is_cuda or state.dtype != torch.float32 or state.dim() != 2 or state.shape[1] < width
+            or state.stride(1) != 1):
+        raise KernelError(f"the recurrent state must be CUDA fp32 [slots][>= {width}], got {tuple(state.shape)}")
+    stride = state.stride(0) if state.shape[0] > 1 else state.shape[1]
+    S = batch.n_segments
+    _i32("seg_start", batch.seg_start, S + 1)
+    _i32("seg_slot", batch.seg_slot, S)
+    ld_out = out_width or width
+    out = torch.empty((T, ld_out), dtype=out_dtype, device=p.device)
+    # the decoding requests at a step's head take one token each; portions of prompts behind them walk
+    singles = S if batch.max_segment == 1 else batch.leading_singles
+    for first, count, longest in ((0, singles, 1), (singles, S - singles, batch.max_segment)):
+        if count > 0:
+            lib.call("fwb_gated_average", ptr(p), c_longlong(columns), int(z_col), int(x_col), int(g_col), ptr(z_bias),
+                     ptr(x_bias), ptr(state), c_longlong(stride), ptr(batch.seg_start), ptr(batch.seg_slot), first, count,
+                     longest, ptr(out), is_bf16(out), width, ld_out, stream())
+    return out
+
+
+def place_heads_(o: torch.Tensor, heads: int, head_dim: int, channels: int, out: torch.Tensor, col0: int, width: int,
+                 scale: float = 1.0, positions: Optional[torch.Tensor] = None, table: Optional[torch.Tensor] = None,
+                 pairing: str = "interleaved") -> torch.Tensor:
+    """``out[t][col0 + h channels + c] = scale * turn(o[t][h])[c]``: the first ``channels`` of every head of
+    ``o`` ([T][heads head_dim]), side by side, turned back by the token's position when a ``table`` ([positions]
+    [rot/2][2]) is given.  The columns behind the heads up to ``col0 + width`` hold ``scale`` in two halves (its
+    value in the row's dtype, and the rest) and then zeros: a product whose matrix has a bias vector in both
+    adds ``scale * bias``."""
+    from .ops import ROPE_PAIRINGS
+    check_tensor("head outputs", o)
+    check_tensor("placed rows", out, o.dtype)
+    T = o.shape[0]
+    if o.shape[1] != heads * head_dim or out.shape[0] != T or col0 < 0 or col0 + width > out.shape[1]:
+        raise KernelError("the heads and the columns they are placed in do not fit")
+    rot = 0
+    if table is not None:
+        check_tensor("rotation table", table, torch.float32)
+        _i32("positions", positions, T)
+        rot = 2 * table.shape[1]
+    lib.call("fwb_place_heads", ptr(o), ptr(positions) if rot else None, ptr(table) if rot else None, rot,
+             ROPE_PAIRINGS[pairing], c_float(scale), out.data_ptr() + col0 * out.element_size(),
+             c_longlong(out.shape[1]), is_bf16(out), T, heads, head_dim, channels, width, stream())
+    return out

@@ -252,7 +252,9 @@ def qk_norm_rope(qkv: torch.Tensor, q_norm: Optional[torch.Tensor], k_norm: Opti
                  block_table: Optional[torch.Tensor], k_pool: Optional[torch.Tensor],
                  v_pool: Optional[torch.Tensor], n_heads: int, n_kv_in: int, head_dim: int,
                  rotary_dim: int, eps: float, q_dtype: torch.dtype, pairing: str = "half_split",
-                 unit_rms_after: bool = False, norm_dim: int = 0) -> torch.Tensor:
+                 unit_rms_after: bool = False, norm_dim: int = 0, bias: Optional[torch.Tensor] = None,
+                 temp: Optional[torch.Tensor] = None, value_table: Optional[torch.Tensor] = None,
+                 value_rotary: int = 0) -> torch.Tensor:
     """Per-head RMSNorm + RoPE of q and k, k/v written to their pages; returns q [T][nh*hd].
 
     ``unit_rms_after``: instead of the weighted norm in front of the rotation, every head of q and k
@@ -263,16 +265,30 @@ def qk_norm_rope(qkv: torch.Tensor, q_norm: Optional[torch.Tensor], k_norm: Opti
     ``n_kv_in`` is the number of KV heads present in ``qkv`` (0: queries only).
     ``table`` is [max_pos][rotary_dim/2][2] fp32 (cos, sin); pair i turns by entry i.
     ``pairing``: which two channels pair i is made of -- "half_split" (i, i + rotary_dim/2) or
-    "interleaved" (2i, 2i + 1)."""
+    "interleaved" (2i, 2i + 1).
+
+    ``qkv`` may be the first columns of a wider buffer.  ``bias``: fp32 [columns of q|k|v], added to the
+    projection first; ``temp``: fp32 [n_heads], multiplies the finished query of its head;
+    ``value_rotary`` > 0: the first that many channels of every value head turn by their own position as
+    well, by ``value_table`` ([max_pos][value_rotary/2][2]) with the same pairing, before they are stored."""
     try:
         pairing_code = ROPE_PAIRINGS[pairing]
     except KeyError:
         raise KernelError(f"unknown rotary pairing {pairing!r}; known: " + ", ".join(ROPE_PAIRINGS)) from None
-    check_tensor("qkv", qkv)
+    width = (n_heads + 2 * n_kv_in) * head_dim
+    if not qkv.is_cuda or qkv.dim() != 2 or qkv.stride(1) != 1:
+        raise KernelError("qkv must be a CUDA matrix with contiguous rows")
     T = qkv.shape[0]
-    if qkv.shape[1] != (n_heads + 2 * n_kv_in) * head_dim:
-        raise KernelError(f"qkv has {qkv.shape[1]} columns, expected "
-                          f"{(n_heads + 2 * n_kv_in) * head_dim}")
+    if qkv.shape[1] != width:
+        raise KernelError(f"qkv has {qkv.shape[1]} columns, expected {width}")
+    if bias is not None:
+        check_tensor("q|k|v bias", bias, torch.float32, (width,))
+    if temp is not None:
+        check_tensor("head factors", temp, torch.float32, (n_heads,))
+    if value_rotary:
+        check_tensor("value table", value_table, torch.float32)
+        if value_rotary % 2 or value_rotary > head_dim or tuple(value_table.shape[1:]) != (value_rotary // 2, 2):
+            raise KernelError("value table must be [positions][value_rotary/2][2]")
     check_tensor("rope table", table, torch.float32)
     if table.dim() != 3 or table.shape[1] != max(1, rotary_dim // 2) or table.shape[2] != 2:
         raise KernelError("rope table must be [positions][rotary_dim/2][2]")
@@ -302,17 +318,19 @@ def qk_norm_rope(qkv: torch.Tensor, q_norm: Optional[torch.Tensor], k_norm: Opti
              ptr(k_norm if use_norm == 1 else None), ptr(table),
              ptr(positions), ptr(tok_seg), ptr(block_table), max_pages, page_size, ptr(q_out),
              is_bf16(q_out), ptr(k_pool), ptr(v_pool), cache_bf16, T, n_heads, n_kv_in, head_dim,
-             rotary_dim, c_float(eps), use_norm, pairing_code, int(norm_dim), stream())
+             rotary_dim, c_float(eps), use_norm, pairing_code, int(norm_dim), c_longlong(qkv.stride(0) if T > 1 else width),
+             ptr(bias), ptr(temp), ptr(value_table) if value_rotary else None, int(value_rotary), stream())
     return q_out
 
 
 def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
                    positions: torch.Tensor, tok_seg: torch.Tensor, block_table: torch.Tensor,
                    n_heads: int, window: int, scale: float, out_dtype: torch.dtype,
-                   sink: Optional[torch.Tensor] = None, softcap: float = 0.0) -> torch.Tensor:
+                   sink: Optional[torch.Tensor] = None, softcap: float = 0.0, keep_first: int = 0) -> torch.Tensor:
     """Causal GQA over the paged cache, SIMT fp32 arithmetic.  q: [T][nh*hd].  ``sink``: fp32 [nh], a
     score per head that joins every softmax denominator (not scaled, not capped, without a value);
-    ``softcap`` > 0: scores become ``softcap * tanh(score / softcap)`` behind the scale."""
+    ``softcap`` > 0: scores become ``softcap * tanh(score / softcap)`` behind the scale; ``keep_first`` > 0
+    (with a sliding window): the sequence's first that many positions stay visible."""
     check_tensor("q", q)
     check_tensor("k pool", k_pool)
     check_tensor("v pool", v_pool, k_pool.dtype, k_pool.shape)
@@ -331,7 +349,7 @@ def attention_simt(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Tensor,
     lib.call("fwb_attention_simt_sink", ptr(q), is_bf16(q), ptr(k_pool), ptr(v_pool), is_bf16(k_pool),
              ptr(positions), ptr(tok_seg), ptr(block_table), block_table.shape[1], page_size,
              ptr(out), is_bf16(out), T, n_heads, n_kv, head_dim, window, c_float(scale), ptr(sink),
-             c_float(softcap), stream())
+             c_float(softcap), int(keep_first), stream())
     return out
 
 
@@ -356,7 +374,7 @@ def _sink_and_groups(sink, groups, n_heads: int, n_kv: int):
 
 def attention_prefill_mma(q, k_pool, v_pool, positions, seg_start, tile_seg, tile_tok0, n_tiles,
                           tokens_per_tile, block_table, n_heads, window, scale, out=None,
-                          sink=None, groups=None, softcap: float = 0.0) -> torch.Tensor:
+                          sink=None, groups=None, softcap: float = 0.0, keep_first: int = 0) -> torch.Tensor:
     """Causal GQA of prompt portions (any mix of segments) on tensor cores; all bf16.  Only the
     rows of the given tiles are written (``out``: a tensor like q that other rows already live in).
     ``v_pool`` may be ``k_pool`` itself; ``sink``, ``groups``: see ``_sink_and_groups``; ``softcap`` > 0:
@@ -381,7 +399,7 @@ def attention_prefill_mma(q, k_pool, v_pool, positions, seg_start, tile_seg, til
     lib.call("fwb_attention_prefill_mma_capped", ptr(q), ptr(k_pool), ptr(v_pool), ptr(positions),
              ptr(seg_start), ptr(tile_seg), ptr(tile_tok0), ptr(block_table), block_table.shape[1],
              page_size, ptr(out), n_tiles, n_heads, groups, head_dim, tokens_per_tile, window,
-             c_float(scale), ptr(sink), n_kv, c_float(softcap), stream())
+             c_float(scale), ptr(sink), n_kv, c_float(softcap), int(keep_first), stream())
     return out
 
 
@@ -393,7 +411,7 @@ def attention_tcgen05_shape_ok(n_heads: int, n_kv: int, head_dim: int, page_size
 
 def attention_prefill_tcgen05(q, k_pool, v_pool, positions, seg_start, tile_seg, tile_tok0, n_tiles,
                               tokens_per_tile, block_table, n_heads, window, scale, out=None,
-                              sink=None, softcap: float = 0.0) -> torch.Tensor:
+                              sink=None, softcap: float = 0.0, keep_first: int = 0) -> torch.Tensor:
     """The same operation on tcgen05 tensor cores: 128 query rows per CTA, S and PV in tensor
     memory (head sizes 64 and 128); all bf16."""
     check_tensor("q", q, torch.bfloat16)
@@ -416,7 +434,7 @@ def attention_prefill_tcgen05(q, k_pool, v_pool, positions, seg_start, tile_seg,
     lib.call("fwb_attention_prefill_tcgen05_capped", ptr(q), ptr(k_pool), ptr(v_pool), ptr(positions),
              ptr(seg_start), ptr(tile_seg), ptr(tile_tok0), ptr(block_table), block_table.shape[1],
              page_size, num_pages, ptr(out), n_tiles, n_heads, n_kv, head_dim, tokens_per_tile, window,
-             c_float(scale), ptr(sink), c_float(softcap), stream())
+             c_float(scale), ptr(sink), c_float(softcap), int(keep_first), stream())
     return out
 
 
@@ -472,7 +490,8 @@ def set_decode_attention_tma(on: bool, stages: int = 0) -> None:
 
 def attention_decode_mma(q, k_pool, v_pool, positions, tok_seg, block_table, n_heads, window, scale,
                          splits: int, tiles_per_split: int, merge_in_cluster: bool = False,
-                         out=None, n_tokens=None, sink=None, groups=None, softcap: float = 0.0) -> torch.Tensor:
+                         out=None, n_tokens=None, sink=None, groups=None, softcap: float = 0.0,
+                         keep_first: int = 0) -> torch.Tensor:
     """Causal GQA of single decode tokens on tensor cores, the context cut into ``splits``
     slices of ``tiles_per_split`` 64-key tiles that run as separate CTAs and are merged: inside
     the kernel (``merge_in_cluster``, up to 8 slices as a thread-block cluster) or through scratch
@@ -504,6 +523,6 @@ def attention_decode_mma(q, k_pool, v_pool, positions, tok_seg, block_table, n_h
     lib.call("fwb_attention_decode_mma_capped", ptr(q), ptr(k_pool), ptr(v_pool), ptr(positions),
              ptr(tok_seg), ptr(block_table), block_table.shape[1], page_size, k_pool.shape[0], ptr(out), ptr(part_o),
              ptr(part_ml), T, n_heads, groups, head_dim, splits, tiles_per_split, window,
-             c_float(scale), 1 if in_cluster else 0, ptr(sink), n_kv, c_float(softcap), stream(),
+             c_float(scale), 1 if in_cluster else 0, ptr(sink), n_kv, c_float(softcap), int(keep_first), stream(),
              launches=2 if (splits > 1 and not in_cluster) else 1)
     return out

@@ -50,17 +50,26 @@ def delta_rule(p: torch.Tensor, taps: torch.Tensor, a_log: torch.Tensor, dt_bias
     return o
 
 
-def gated_head_norm(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float,
-                    out_dtype: torch.dtype) -> torch.Tensor:
+def gated_head_norm(o: torch.Tensor, gate: torch.Tensor, weight, eps: float, out_dtype: torch.dtype,
+                    out: torch.Tensor = None, col0: int = 0, scale: float = 1.0) -> torch.Tensor:
     """``weight * o / sqrt(mean(o^2) + eps) * silu(gate)`` per (token, head).  o: fp32 [T][H][e];
-    ``gate``: fp32 [T][H e], possibly a view of columns of a wider row-major tensor; weight: fp32 [e]."""
+    ``gate``: fp32 [T][H e], possibly a view of columns of a wider row-major tensor; weight: fp32 [e], or None:
+    every channel counts ``scale``.  ``out``: rows that hold the result from column ``col0`` on (a new
+    [T][H e] otherwise)."""
     check_tensor("recurrence output", o, torch.float32)
     T, H, e = o.shape
     if (not gate.is_cuda or gate.dtype != torch.float32 or tuple(gate.shape) != (T, H * e)
             or gate.stride(1) != 1):
         raise KernelError(f"the gate must be CUDA fp32 [{T}][{H * e}] with contiguous rows")
-    check_tensor("head norm weight", weight, torch.float32, (e,))
-    out = torch.empty((T, H * e), dtype=out_dtype, device=o.device)
-    lib.call("fwb_gated_head_norm", ptr(o), ptr(gate), c_longlong(gate.stride(0)), ptr(weight), c_float(eps),
-             ptr(out), is_bf16(out), T, H, e, stream())
+    if weight is not None:
+        check_tensor("head norm weight", weight, torch.float32, (e,))
+    if out is None:
+        out = torch.empty((T, H * e), dtype=out_dtype, device=o.device)
+    else:
+        check_tensor("normed rows", out, out_dtype)
+        if out.shape[0] != T or col0 < 0 or col0 + H * e > out.shape[1]:
+            raise KernelError("the heads do not fit the columns they are written to")
+    lib.call("fwb_gated_head_norm", ptr(o), ptr(gate), c_longlong(gate.stride(0) if T > 1 else H * e), ptr(weight),
+             c_float(scale), c_float(eps), out.data_ptr() + col0 * out.element_size(), is_bf16(out),
+             c_longlong(out.shape[1]), T, H, e, stream())
     return out

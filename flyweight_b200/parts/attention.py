@@ -14,7 +14,8 @@ import torch
 
 from ..kernels import ops
 from ..weights.loader import TensorDecl
-from .base import FixedState, Mixer, PagedKV, Precision, build_position, register_mixer
+from ..config.spec import PartSpec
+from .base import FixedState, Mixer, PagedKV, PositionEncoding, Precision, build_position, register_mixer
 
 
 @register_mixer("gqa_attention")
@@ -43,7 +44,15 @@ class GQAttention(Mixer):
     sigmoid(g h) of its head; "element": ``g`` [heads value_dim][H], channel by channel; both read the
     mixer's input); ``value_mix`` ("source": this layer's values, as cached, are also handed on to later
     layers of the step under ``value_mix_key``; "mixed": v <- (1 - lam) v + lam v_source with the
-    tensor ``vmix``, one number, before v is cached)."""
+    tensor ``vmix``, one number, before v is cached); ``keep_first`` (n > 0, with a window: the sequence's first n
+    positions stay visible, and their pages are kept); ``bias`` (True: tensors ``q_b``, ``k_b``, ``v_b`` [rows] are
+    added to the projections and ``o_b`` [H] to the output projection); ``temp`` (True: tensor ``temp`` [heads], a
+    number per head on the scores, in front of the cap); ``turned_values`` (True: the value of position j is rotated
+    by j over all its ``value_dim`` channels, with the position part's base and pairing and no scaling, and is cached
+    so; each head's output at position i is turned back by i).
+
+    A mixer without output gate, convolutions, mixed values, a norm over the whole projection or a foreign cache
+    can be one of several on one input (``joins``, see ``Mixer``)."""
     graph_safe = True
     takes_deferred_norm = True
     adds_residual = True
@@ -95,8 +104,34 @@ class GQAttention(Mixer):
             raise ValueError("softcap must not be negative")
         if self.value_dim != self.qk_dim or self.qk_dim % 16:
             self.head_dim = -(-max(self.qk_dim, self.value_dim) // 16) * 16
+        self.keep_first = int(p.get("keep_first", 0) or 0)
+        self.has_bias = bool(p.get("bias", False))
+        self.has_temp = bool(p.get("temp", False))
+        self.turned_values = bool(p.get("turned_values", False))
+        if self.keep_first < 0 or (self.keep_first and not self.window):
+            raise ValueError("kept first positions go with a sliding window")
+        self.value_turn = None
+        if self.turned_values:
+            base = self.params["position"]
+            if "theta" not in base.params:
+                raise ValueError("rotated values take base and pairing from a rotary position part")
+            if self.value_dim % 2:
+                raise ValueError("rotated values need an even value size")
+            self.value_turn = build_position(PartSpec("rope", {
+                "theta": base.params["theta"], "rotary_dim": self.value_dim, "pairing": self.position.pairing}))
+        plain_encode = type(self.position).encode is PositionEncoding.encode
+        extras = self.has_bias or self.has_temp or self.turned_values
+        self.joins = (plain_encode and self.unit_rms_eps is None
+                      and not (self.gate or self.value_mix or self.conv_taps or self.shares_cache
+                               or self.qk_norm == "whole"))
+        if extras and not self.joins:
+            raise ValueError("biases, factors per head and rotated values do not combine with output gates, mixed "
+                             "values, convolutions, a norm over the whole projection, a norm behind the rotation, "
+                             "another's cache or a position encoding of its own kind")
+        # heads leave through ``place_heads_`` (packed, turned back, scaled) in the joined form
+        self._placed = extras
         # the launches LFM2 makes: nothing of the above, so the fused decode kernel and the native plan apply
-        self._plain = not (self.has_sink or self.softcap or self.gate or self.value_mix or self.conv_taps
+        self._plain = not (extras or self.keep_first or self.has_sink or self.softcap or self.gate or self.value_mix or self.conv_taps
                            or self.qk_norm == "whole" or (self.head_dim != self.qk_dim and self.eps is not None))
         # q|k|v leave their product in fp32 when a norm over the whole projection works on them in place before
         # the head kernel reads them: one rounding, not two.  (Mixed values are rounded on both sides of the
@@ -106,7 +141,7 @@ class GQAttention(Mixer):
         # buffer of its own, so the gate's columns stay where the product left them)
         self._gate_in_projection = self.gate == "head" and self.conv_taps > 0
         self.w_qkv = self.w_o = self.q_norm = self.k_norm = self.w_gate = self.sink = self.vmix = None
-        self.taps = None
+        self.taps = self.qkv_bias = self.temp = None
 
     @property
     def _kv_in(self) -> int:
@@ -135,9 +170,53 @@ class GQAttention(Mixer):
             out[n["g"]] = TensorDecl((self.n_heads * (self.value_dim if self.gate == "element" else 1), H))
         if self.value_mix == "mixed":
             out[n["vmix"]] = TensorDecl((), "bias", also=((1,),))
+        if self.has_bias:
+            out[n["q_b"]] = TensorDecl((self.n_heads * hd,), "bias")
+            out[n["k_b"]] = TensorDecl((self.n_kv * hd,), "bias")
+            out[n["v_b"]] = TensorDecl((self.n_kv * self.value_dim,), "bias")
+            out[n["o_b"]] = TensorDecl((H,), "bias")
+        if self.has_temp:
+            out[n["temp"]] = TensorDecl((self.n_heads,), "norm")
         return out
 
+    @property
+    def out_width(self) -> int:
+        """Columns this mixer fills of a joined output row: its heads side by side, with a bias two more for
+        the constant that carries it, rounded up to what the products' tiles take."""
+        used = self.n_heads * self.value_dim + (2 if self.has_bias else 0)
+        return -(-used // 8) * 8
+
+    def _output_columns(self, get):
+        """[H][out_width]: the output matrix for rows that ``place_heads_`` made; the bias stands in the two
+        columns behind the heads', which meet the row's constant (its value and what rounding left of it)."""
+        w_o = get(self.names["o"])
+        wide = w_o.new_zeros((w_o.shape[0], self.out_width))
+        used = self.n_heads * self.value_dim
+        wide[:, :used] = w_o
+        if self.has_bias:
+            bias = get(self.names["o_b"])
+            if bias.dtype != w_o.dtype:
+                wide, bias = wide.to(torch.float32), bias.to(torch.float32)
+            wide[:, used] = bias
+            wide[:, used + 1] = bias
+        return wide
+
     def bind(self, get, precision: Precision, device):
+        self.w_qkv = precision.matrix(self._bind_inner(get, precision, device), device)
+        w_o = self._output_columns(get) if self._placed else get(self.names["o"])
+        D = self.head_dim
+        if not self._placed and self.value_dim != D:      # zero columns where the padded channels of a head arrive
+            wide = w_o.new_zeros((w_o.shape[0], self.n_heads, D))
+            wide[:, :, :self.value_dim] = w_o.view(w_o.shape[0], self.n_heads, self.value_dim)
+            w_o = wide.view(w_o.shape[0], self.n_heads * D)
+        self.w_o = precision.matrix(w_o, device)
+
+    def bind_joined(self, get, precision: Precision, device):
+        """Binds everything but the two products' matrices and returns those, still as stored: rows of the
+        input projection, columns of the output projection."""
+        return self._bind_inner(get, precision, device), self._output_columns(get)
+
+    def _bind_inner(self, get, precision: Precision, device):
         n = self.names
         D = self.head_dim
 
@@ -162,13 +241,7 @@ class GQAttention(Mixer):
         if len(dtypes) > 1:
             mats = [m.to(torch.float32) for m in mats]
         # one projection for q|k|v (|gate): the rows of the matrices, one after the other
-        self.w_qkv = precision.matrix(torch.cat(mats, dim=0), device)
-        w_o = get(n["o"])
-        if self.value_dim != D:                   # zero columns where the padded channels of a head arrive
-            wide = w_o.new_zeros((w_o.shape[0], self.n_heads, D))
-            wide[:, :, :self.value_dim] = w_o.view(w_o.shape[0], self.n_heads, self.value_dim)
-            w_o = wide.view(w_o.shape[0], self.n_heads * D)
-        self.w_o = precision.matrix(w_o, device)
+        rows = torch.cat(mats, dim=0)
         def channels_padded(vector, per_head):
             """[heads * per_head] -> [heads * D]: zeros behind every head's own channels."""
             if per_head == D:
@@ -196,11 +269,18 @@ class GQAttention(Mixer):
                                            device)
         if self.value_mix == "mixed":
             self.vmix = precision.vector(get(n["vmix"]).reshape(1), device)
+        if self.has_bias:
+            self.qkv_bias = precision.vector(torch.cat([
+                channels_padded(get(n[name]).reshape(-1), per) for name, per in
+                (("q_b", self.qk_dim), ("k_b", self.qk_dim), ("v_b", self.value_dim))]), device)
+        if self.has_temp:
+            self.temp = precision.vector(get(n["temp"]), device)
+        return rows
 
     def _matrices(self):
         return tuple(m for m in (self.w_qkv, self.w_o, self.w_gate) if m is not None)
 
-    def weight_bytes(self):
+    def weight_bytes(self):                       # (0 while the matrices belong to the mixer that joined this one)
         return sum(m.numel() * m.element_size() for m in self._matrices())
 
     def flops_per_token(self):
@@ -208,7 +288,7 @@ class GQAttention(Mixer):
 
     def context_flops(self, n_tokens):
         # QK^T and PV: 4 operations per (query, visible key, channel); half the pairs are masked
-        if self.window and n_tokens > self.window:
+        if self.window and n_tokens > self.window:      # (kept first positions: a handful of keys more)
             pairs = n_tokens * self.window - 0.5 * self.window * self.window
             return 4.0 * pairs * self.n_heads * self.head_dim
         if self.chunk and n_tokens > self.chunk:
@@ -228,7 +308,7 @@ class GQAttention(Mixer):
         return {"unit_rms_after": True, "norm_dim": self.qk_dim}
 
     def state_spec(self):
-        paged = None if self.shares_cache else PagedKV(self.n_kv, self.head_dim, self.window)
+        paged = None if self.shares_cache else PagedKV(self.n_kv, self.head_dim, self.window, self.keep_first)
         if self.conv_taps > 1:
             channels = (self.n_heads + 2 * self._kv_in) * self.head_dim
             rolling = FixedState((self.conv_taps - 1, channels))
@@ -237,9 +317,19 @@ class GQAttention(Mixer):
 
     def prepare(self, max_positions, device):
         self.position.prepare(max_positions, device)
+        if self.value_turn is not None:
+            if getattr(self.position, "rotary_dim", 0) == self.value_dim and not self.params["position"].params.get("scaling"):
+                self.value_turn._table = self.position._table         # the keys' own angles: one table
+            else:
+                self.value_turn.prepare(max_positions, device)
 
     def forward(self, ctx, h, cache, residual=None):
         act = ctx.precision.act_dtype
+        if self._placed:
+            p = ops.linear(h, self.w_qkv, torch.float32)
+            rows = torch.empty((p.shape[0], self.out_width), dtype=act, device=p.device)
+            self.forward_joined(ctx, p, 0, cache, rows, 0, 1.0)
+            return ops.linear_into_residual(rows, self.w_o, residual)
         if not self._plain:
             return self._forward_general(ctx, h, cache, residual)
         # q|k|v in the activation dtype; the head norm and the rotation widen it to fp32
@@ -263,6 +353,25 @@ class GQAttention(Mixer):
         out = attention_kernels.paged_attention(ctx, q, cache, block_table, self.n_heads,
                                                 self.span, self.scale, act)
         return ops.linear_into_residual(out, self.w_o, residual)
+
+    def forward_joined(self, ctx, p, col0, cache, rows, out_col, scale):
+        """Everything between the two products: ``p`` holds this mixer's projections (fp32) from column ``col0``
+        on, its ``out_width`` columns of ``rows`` from ``out_col`` on receive the heads' outputs times ``scale``."""
+        from ..kernels import attention as attention_kernels
+        from ..kernels import mixing
+        D = self.head_dim
+        qkv = p[:, col0:col0 + (self.n_heads + 2 * self.n_kv) * D]
+        block_table = ctx.batch.block_tables[cache.group]
+        turn = self.value_turn._table if self.value_turn is not None else None
+        q = self.position.encode(ctx, qkv, n_heads=self.n_heads, n_kv_in=self.n_kv, head_dim=D, q_norm=self.q_norm,
+                                 k_norm=self.k_norm, eps=self.eps, cache=cache, block_table=block_table,
+                                 bias=self.qkv_bias, temp=self.temp, value_table=turn,
+                                 value_rotary=self.value_dim if turn is not None else 0, **self._encode_extra())
+        out = attention_kernels.paged_attention(ctx, q, cache, block_table, self.n_heads, self.span, self.scale,
+                                                ctx.precision.act_dtype, sink=self.sink, softcap=self.softcap,
+                                                keep_first=self.keep_first)
+        mixing.place_heads_(out, self.n_heads, D, self.value_dim, rows, out_col, self.out_width, scale,
+                            ctx.batch.positions, turn, self.position.pairing)
 
     def _forward_general(self, ctx, h, cache, residual=None):
         """The mixer with any of: a norm over the whole projection, padded heads under a weighted norm,
@@ -308,7 +417,8 @@ class GQAttention(Mixer):
                                  eps=None if whole else (self.eps if self.unit_rms_eps is None else self.unit_rms_eps),
                                  cache=cache, block_table=block_table, **extra)
         out = attention_kernels.paged_attention(ctx, q, cache, block_table, self.n_heads, self.span, self.scale,
-                                                act, sink=self.sink, softcap=self.softcap)
+                                                act, sink=self.sink, softcap=self.softcap,
+                                                keep_first=self.keep_first)
         if self._gate_in_projection:
             mixing.sigmoid_gate_cols_mul_(out, projected, self._qkv_columns, self.n_heads, D)
         elif self.gate:
@@ -319,8 +429,8 @@ class GQAttention(Mixer):
         """The same operations for the native step plan (``engine/plan.py``)."""
         from ..engine.plan import EPI_ACT, NotPlannable
         if not self._plain:
-            raise NotPlannable("sinks, capped scores, gates, mixed values and norms over the whole projection "
-                               "have no native plan form")
+            raise NotPlannable("biases, factors per head, rotated values, kept first positions, sinks, capped scores, "
+                               "gates, mixed values and norms over the whole projection have no native plan form")
         act = builder.act_dtype
         plan_position = getattr(self.position, "plan", None)
         if self.unit_rms_eps is not None:

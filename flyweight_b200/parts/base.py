@@ -18,6 +18,11 @@ Interfaces
 ``Mixer.forward(ctx, h, cache)`` -> fp32 [T][H]
     h: normalised input; cache: the ``LayerCache`` the manager made for this
     execution (or for the execution it shares with).  Returns the residual delta.
+``Mixer.joins``  (False: no)
+    whether the mixer can be one of several on one input: ``bind_joined`` binds its vectors and hands out the
+    rows of its input projection and the columns of its output projection, and ``forward_joined(ctx, p, col0,
+    cache, rows, out_col, scale)`` does what lies between the two products, from its columns of a shared fp32
+    projection to its ``out_width`` columns of a shared row.
 ``FeedForward.forward(ctx, h)`` -> fp32 [T][H]
     A mixer or feed-forward with ``adds_residual`` is called with ``residual=x`` as well and
     may add its delta into x itself (its last product's epilogue); it then returns None.
@@ -84,10 +89,12 @@ class Precision:
 @dataclass(frozen=True)
 class PagedKV:
     """Keys and values that grow with the sequence.  ``window`` > 0: only the last
-    ``window`` positions are ever read again, older pages may be given back."""
+    ``window`` positions (and the sequence's first ``keep_first``) are ever read again, the pages between them
+    may be given back."""
     n_kv_heads: int
     head_dim: int
     window: int = 0
+    keep_first: int = 0        # with a window: the first that many positions are read for as long as the request lives
     values: bool = True        # False: one pool only (a latent row per token serves as key and value)
 
 
@@ -191,12 +198,14 @@ class PositionEncoding(Part):
                        else torch.zeros((1, 1, 2), dtype=torch.float32, device=device))
 
     def encode(self, ctx, qkv, *, n_heads: int, n_kv_in: int, head_dim: int, q_norm, k_norm,
-               eps: float, cache, block_table, unit_rms_after: bool = False, norm_dim: int = 0):
+               eps: float, cache, block_table, unit_rms_after: bool = False, norm_dim: int = 0, bias=None,
+               temp=None, value_table=None, value_rotary: int = 0):
         """qkv: [T][(n_heads + 2 n_kv_in) head_dim] in the activation dtype (``n_kv_in`` 0: queries
         only, for a mixer that reads another execution's cache).  Returns q [T][n_heads head_dim].
         ``unit_rms_after`` (only handed over when set): no weighted norm in front of the rotation;
         every head of q and k is brought to unit root mean square behind it, the mean taken over the
-        head's first ``norm_dim`` channels (the rest is zero padding)."""
+        head's first ``norm_dim`` channels (the rest is zero padding).  ``bias``, ``temp``, ``value_table`` and
+        ``value_rotary`` (only handed over when set): see ``ops.qk_norm_rope``."""
         from ..kernels import ops
         batch = ctx.batch
         return ops.qk_norm_rope(
@@ -204,7 +213,8 @@ class PositionEncoding(Part):
             block_table if n_kv_in else None, cache.k_pool if n_kv_in else None,
             cache.v_pool if n_kv_in else None, n_heads, n_kv_in, head_dim, self.rotary_dim,
             float(eps or 0.0), ctx.precision.act_dtype, pairing=self.pairing,
-            unit_rms_after=unit_rms_after, norm_dim=norm_dim)
+            unit_rms_after=unit_rms_after, norm_dim=norm_dim, bias=bias, temp=temp, value_table=value_table,
+            value_rotary=value_rotary)
 
     def rotation(self):
         """(table, rotary_dim, pairing) for a mixer that can do the default ``encode`` inside a kernel
@@ -227,6 +237,8 @@ class PositionEncoding(Part):
 
 
 class Mixer(Part):
+    joins: bool = False
+
     def state_spec(self):
         return None
 

@@ -1,11 +1,12 @@
-"""Mixture-of-experts feed-forward with a grouped, bias-corrected softmax router and identity experts.
+"""Mixture-of-experts feed-forward with a router (grouped, bias-corrected) and identity experts.
 
-Router scores s = softmax(W_router h) over all router outputs, in fp32.  The choice is made on s +
-correction: the outputs form ``groups`` equal runs of neighbours, only the ``keep_groups`` runs with
+Router scores s = softmax(W_router h) over all router outputs, or the sigmoid of each, in fp32.  The choice is
+made on s + correction (no correction: on s): the outputs form ``groups`` equal runs of neighbours, only the ``keep_groups`` runs with
 the largest choice value stay in the race, and the ``top`` largest survivors are chosen; the weights
 are the plain s of the chosen, not renormalised.  The first ``experts`` outputs are small gated
 feed-forwards, down(act(gate h) * (up h)); the ``identity`` outputs behind them hand h itself on.  The
-result is the weighted sum over the chosen.
+result is the weighted sum over the chosen; a model may instead put the weight on what an expert reads,
+sum of expert(s h) over the chosen.
 """
 from __future__ import annotations
 
@@ -20,8 +21,8 @@ from .base import FeedForward, Precision, register_feed_forward
 @register_feed_forward("routed_experts")
 class RoutedExperts(FeedForward):
     """params: hidden_size, ffn_dim (of one expert), experts, identity (0), top, groups (1), keep_groups
-    (1), activation ("silu").  tensors: router [experts + identity][H], correction [experts + identity],
-    and per expert j ``gate{j}``, ``up{j}`` [F][H], ``down{j}`` [H][F]."""
+    (1), activation ("silu"), scores ("softmax" | "sigmoid"), corrected (True), weights_on ("output" | "input").
+    tensors: router [experts + identity][H], correction [experts + identity] (unless ``corrected`` is False), and per expert j ``gate{j}``, ``up{j}`` [F][H], ``down{j}`` [H][F]."""
     graph_safe = True
 
     def __init__(self, spec):
@@ -35,6 +36,13 @@ class RoutedExperts(FeedForward):
         self.groups = int(p.get("groups", 1) or 1)
         self.keep_groups = int(p.get("keep_groups", self.groups) or self.groups)
         self.activation = str(p.get("activation", "silu"))
+        self.scores = str(p.get("scores", "softmax"))
+        self.corrected = bool(p.get("corrected", True))
+        self.weights_on = str(p.get("weights_on", "output"))
+        if self.scores not in expert_kernels.ROUTER_SCORES:
+            raise ValueError(f"unknown router scores {self.scores!r}; known: " + ", ".join(expert_kernels.ROUTER_SCORES))
+        if self.weights_on not in ("output", "input"):
+            raise ValueError(f"expert weights go on the output or on the input, not on {self.weights_on!r}")
         outputs = self.n_experts + self.n_identity
         if self.activation not in ops.GATE_ACTIVATIONS:
             raise ValueError(f"unknown gate activation {self.activation!r}")
@@ -53,7 +61,9 @@ class RoutedExperts(FeedForward):
 
     def declare(self):
         n, H, F = self.names, self.hidden, self.ffn_dim
-        out = {n["router"]: TensorDecl((self.n_outputs, H)), n["correction"]: TensorDecl((self.n_outputs,), "bias")}
+        out = {n["router"]: TensorDecl((self.n_outputs, H))}
+        if self.corrected:
+            out[n["correction"]] = TensorDecl((self.n_outputs,), "bias")
         for j in range(self.n_experts):
             out[n[f"gate{j}"]] = TensorDecl((F, H))
             out[n[f"up{j}"]] = TensorDecl((F, H))
@@ -64,7 +74,8 @@ class RoutedExperts(FeedForward):
         n = self.names
         # the router runs in fp32 whatever the precision (a bfloat16 matrix widens exactly)
         self.router = precision.vector(get(n["router"]), device)
-        self.correction = precision.vector(get(n["correction"]), device)
+        if self.corrected:
+            self.correction = precision.vector(get(n["correction"]), device)
         mats = [get(n[f"{role}{j}"]) for j in range(self.n_experts) for role in ("gate", "up", "down")]
         dtype = torch.float32 if (precision.name == "float32" or len({m.dtype for m in mats}) > 1) \
             else (mats[0].dtype if mats else precision.act_dtype)
@@ -94,11 +105,12 @@ class RoutedExperts(FeedForward):
         return 2.0 * self.router.numel() + 2.0 * self.top * 3 * self.ffn_dim * self.hidden
 
     def forward(self, ctx, h, add_normed_into=None):
-        ids, weights = expert_kernels.route(h, self.router, self.correction, self.groups, self.keep_groups, self.top)
+        ids, weights = expert_kernels.route(h, self.router, self.correction, self.groups, self.keep_groups, self.top,
+                                            self.scores)
         if h.dtype != self.w_gate_up.dtype:
             h = ops.cast(h, self.w_gate_up.dtype)
         return expert_kernels.experts_forward(h, ids, weights, self.w_gate_up, self.w_down, self.activation,
-                                              add_normed_into)
+                                              add_normed_into, weights_on=self.weights_on)
 
     def forward_add_normed(self, ctx, h, x, norm_weight, eps):
         """``x += norm_weight * unit(ff(h))`` with the weighted sum, the output norm and the residual sum in

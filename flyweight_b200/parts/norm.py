@@ -15,22 +15,25 @@ from .base import DeferredNorm, Norm, Precision, register_norm
 class RMSNorm(Norm):
     """params: size, eps, and optionally ``gain``: one constant that multiplies the normed rows beside the
     weight (a model that adds ``m * norm(y)`` into its stream names m here; it is folded into the weight
-    once, in fp32, when the weight is bound).  tensors: weight [size]."""
+    once, in fp32, when the weight is bound) and ``offset``: added to the stored weight (1 for a model that stores
+    its weights around zero; folded the same way, before the gain).  tensors: weight [size]."""
     graph_safe = True
-
 
     def __init__(self, spec):
         super().__init__(spec)
         self.size = int(self.params["size"])
         self.eps = float(self.params["eps"])
         self.gain = float(self.params.get("gain", 1.0))
+        self.offset = float(self.params.get("offset", 0.0))
         self.weight = None
 
     def declare(self):
-        return {self.names["weight"]: TensorDecl((self.size,), "norm")}
+        return {self.names["weight"]: TensorDecl((self.size,), "bias" if self.offset else "norm")}
 
     def bind(self, get, precision: Precision, device):
         self.weight = precision.vector(get(self.names["weight"]), device)
+        if self.offset:
+            self.weight = (self.weight + self.offset).contiguous()
         if self.gain != 1.0:
             self.weight = (self.weight * self.gain).contiguous()
 
