@@ -141,6 +141,30 @@ def fobatar_like(lfm2: dict, ff: int) -> dict:
             "layers": layers}
 
 
+def vugipel_like(lfm2: dict, ff: int) -> dict:
+    """A Vugipel configuration with the layer sizes of an LFM2 one (width, depth, vocabulary, query and
+    key/value heads of 64): where LFM2 attends, attention inside a window of 1,024 positions with the first
+    16 kept (rotated keys and values, scores capped at 30) beside a retention (width / 128 heads of 128 x 128
+    state); where it has a short convolution, a minGRU of the model's width.  Every layer has routed experts
+    that use as much of the feed-forward per token as LFM2's (32 experts of ff / 8, eight a token)."""
+    width, heads, kv = lfm2["hidden_size"], lfm2["num_attention_heads"], lfm2["num_key_value_heads"]
+    linear_heads = width // 128
+    decay = [round(1.0 - 2.0 ** (-5.0 - 5.0 * h / max(linear_heads - 1, 1)), 6) for h in range(linear_heads)]
+    mlp = {"kind": "moe", "expert": {"ff": ff // 8}, "router": {"experts": 32, "top": 8}}
+    layers = []
+    for index in range(lfm2["num_hidden_layers"]):
+        if index in lfm2["full_attn_idxs"]:
+            left = {"heads": heads, "kv_heads": kv, "dim": 64, "vdim": 64, "scale": 0.125, "softcap": 30.0,
+                    "mask": {"size": 1024, "keep_first": 16}, "rot": {"base": 1000000.0, "dims": 64}}
+            right = {"heads": linear_heads, "dim": 128, "vdim": 128, "decay": decay}
+            mixer = {"left": left, "right": right, "left_scale": 0.7, "right_scale": 0.7}
+            layers.append({"type": "parallel", "mixer": mixer, "mlp": mlp})
+        else:
+            layers.append({"type": "mingru", "mixer": {"width": width}, "mlp": mlp})
+    return {"architecture": "Vugipel", "vocab": lfm2["vocab_size"], "width": width, "norm": {"eps": 1e-5},
+            "layers": layers}
+
+
 # Kemitar, Diforax and Gukosun beside LFM2 at equal layer sizes (--compare): the feed-forward widths are what
 # LFM2's rule makes of ``intermediate_size`` at these sizes.
 KEMITAR = {"kemitar-350m": ("lfm2-350m", 4608), "kemitar-1.2b": ("lfm2-1.2b", 8192)}
@@ -157,7 +181,12 @@ for _name, (_twin, _ff) in GUKOSUN.items():
 FOBATAR = {"fobatar-350m": ("diforax-350m", 4608), "fobatar-1.2b": ("diforax-1.2b", 8192)}
 for _name, (_twin, _ff) in FOBATAR.items():
     MODELS[_name] = fobatar_like(MODELS["lfm2" + _name[len("fobatar"):]], _ff)
-COMPARE = {**KEMITAR, **DIFORAX, **GUKOSUN, **FOBATAR}
+# Vugipel beside Gukosun, the closest model the engine has (windowed attention with capped scores, an attention
+# beside a decayed linear attention), at equal layer sizes; its experts' products are Diforax's
+VUGIPEL = {"vugipel-350m": ("gukosun-350m", 4608), "vugipel-1.2b": ("gukosun-1.2b", 8192)}
+for _name, (_twin, _ff) in VUGIPEL.items():
+    MODELS[_name] = vugipel_like(MODELS["lfm2" + _name[len("vugipel"):]], _ff)
+COMPARE = {**KEMITAR, **DIFORAX, **GUKOSUN, **FOBATAR, **VUGIPEL}
 
 
 def vocab_of(config: dict) -> int:
@@ -293,7 +322,7 @@ def cache_bytes_read(model, context: int) -> int:
         for member in (spec if isinstance(spec, tuple) else (spec,)):
             if member is not None and hasattr(member, "n_kv_heads"):
                 pools = 2 if getattr(member, "values", True) else 1
-                positions = min(seen, member.window) if member.window else seen
+                positions = min(seen, member.window + member.keep_first) if member.window else seen
                 total += positions * pools * member.n_kv_heads * member.head_dim * model.precision.cache_dtype.itemsize
     return total
 
@@ -551,8 +580,9 @@ def run_sizes(args) -> int:
 
 
 def run_compare(args) -> int:
-    """``--compare kemitar-350m|kemitar-1.2b|diforax-350m|diforax-1.2b|gukosun-350m|gukosun-1.2b|fobatar-350m|fobatar-1.2b``: the model with
-    random weights beside its twin (LFM2; for Fobatar, Diforax) at equal layer sizes, both through the same step function -- prompts of 512, 2,048 and 8,192 tokens in one step
+    """``--compare kemitar-350m|kemitar-1.2b|diforax-350m|diforax-1.2b|gukosun-350m|gukosun-1.2b|fobatar-350m|fobatar-1.2b|
+    vugipel-350m|vugipel-1.2b``: the model with random weights beside its twin (LFM2; for Fobatar, Diforax; for
+    Vugipel, Gukosun) at equal layer sizes, both through the same step function -- prompts of 512, 2,048 and 8,192 tokens in one step
     (tokens/s and TFLOP/s of the model's own flop count) and decode steps at batch 1, 8 and 64 over 4,096
     cached tokens (tokens/s, and the bytes a step must read against the measured copy bandwidth).  One
     JSON line per model; the LFM2 line's ffn width is checked to be the one the Kemitar twin was given."""
@@ -881,7 +911,7 @@ def main() -> int:
                              "requests, 256 new tokens each, through the public runtime (e.g. lfm2-350m)")
     parser.add_argument("--compare", default=None, metavar="MODEL",
                         help="kemitar-350m, kemitar-1.2b, diforax-350m, diforax-1.2b, gukosun-350m or gukosun-1.2b beside LFM2, "
-                             "fobatar-350m or fobatar-1.2b beside Diforax, at equal layer sizes: prompts and decode steps")
+                             "fobatar-350m or fobatar-1.2b beside Diforax, vugipel-350m or vugipel-1.2b beside Gukosun, at equal layer sizes: prompts and decode steps")
     parser.add_argument("--kernel-times", default=None, metavar="[MODEL:]decode[@BATCHxCONTEXT]|prefill|TOKENS",
                         help="one step with CUDA events around every launch: time per kernel as JSON")
     args = parser.parse_args()

@@ -25,6 +25,7 @@ namespace {
 
 constexpr int WARPS = 16;
 constexpr int TOKENS = 8;                     // tokens a warp
+template <typename TO> constexpr bool quick() { return sizeof(TO) == 2; }
 constexpr int STRETCH = WARPS * TOKENS;       // tokens a CTA and round
 
 template <int VEC> struct Pack { float v[VEC]; };
@@ -64,17 +65,23 @@ __device__ __forceinline__ void store_vec(__nv_bfloat16* at, const Pack<VEC>& r)
     }
 }
 
-// keep = 1 - sigmoid(z) and add = sigmoid(z) * candidate(u): neither loses digits where the gate is near 0 or 1
+// keep = 1 - sigmoid(z) and add = sigmoid(z) * candidate(u): neither loses digits where the gate is near 0 or 1.
+// QUICK (the serving precision): the exponential and the reciprocal of the special-function unit, fp32 with an
+// error of a few units in the last place; else expf and a division.
+template <bool QUICK>
 __device__ __forceinline__ void gates(float z, float u, float& keep, float& add) {
-    const float e = expf(-fabsf(z)), r = 1.0f / (1.0f + e);
-    const float open = z >= 0.0f ? r : e * r;
-    keep = z >= 0.0f ? e * r : r;
-    float c = u + 0.5f;
-    if (u < 0.0f) {
-        const float f = expf(u);
-        c = f / (1.0f + f);
-    }
-    add = open * c;
+    const float e = QUICK ? __expf(-fabsf(z)) : expf(-fabsf(z));
+    const float r = QUICK ? __fdividef(1.0f, 1.0f + e) : 1.0f / (1.0f + e);
+    const float er = e * r;
+    const float open = z >= 0.0f ? r : er;
+    keep = z >= 0.0f ? er : r;
+    const float f = QUICK ? __expf(fminf(u, 0.0f)) : expf(fminf(u, 0.0f));
+    const float low = QUICK ? __fdividef(f, 1.0f + f) : f / (1.0f + f);
+    add = open * (u < 0.0f ? low : u + 0.5f);
+}
+template <bool QUICK>
+__device__ __forceinline__ float gate_out(float g) {
+    return QUICK ? __fdividef(g, 1.0f + __expf(-g)) : silu_f32(g);
 }
 
 struct Shape {
@@ -113,16 +120,16 @@ gated_average_step_kernel(const Shape sh, TO* __restrict__ out) {
 #pragma unroll
     for (int j = 0; j < VEC; ++j) {
         float keep, add;
-        gates(z.v[j] + (sh.z_bias ? sh.z_bias[c + j] : 0.0f), u.v[j] + (sh.x_bias ? sh.x_bias[c + j] : 0.0f), keep, add);
+        gates<quick<TO>()>(z.v[j] + (sh.z_bias ? sh.z_bias[c + j] : 0.0f), u.v[j] + (sh.x_bias ? sh.x_bias[c + j] : 0.0f), keep, add);
         s.v[j] = fmaf(keep, s.v[j], add);
-        y.v[j] = s.v[j] * silu_f32(g.v[j]);
+        y.v[j] = s.v[j] * gate_out<quick<TO>()>(g.v[j]);
     }
     store_vec<VEC>(mine, s);
     store_vec<VEC>(dst, y);
 }
 
 template <int VEC, typename TO>
-__global__ void __launch_bounds__(WARPS * 32, 1)
+__global__ void __launch_bounds__(WARPS * 32, 2)
 gated_average_walk_kernel(const Shape sh, TO* __restrict__ out) {
     fwb::pdl_entry();
     constexpr int COLS = 32 * VEC;
@@ -146,7 +153,7 @@ gated_average_walk_kernel(const Shape sh, TO* __restrict__ out) {
     int parity = 0;
     for (int base = first; base < last; base += ranks * STRETCH, parity ^= 1) {
         const int t0 = base + rank * STRETCH + warp * TOKENS;
-        Pack<VEC> a[TOKENS], b[TOKENS], g[TOKENS];
+        Pack<VEC> a[TOKENS], b[TOKENS];
 #pragma unroll
         for (int i = 0; i < TOKENS; ++i) {
             const bool on = live && t0 + i < last;
@@ -154,10 +161,9 @@ gated_average_walk_kernel(const Shape sh, TO* __restrict__ out) {
             if (on) {
                 a[i] = load_vec<VEC>(row + sh.z_col);
                 b[i] = load_vec<VEC>(row + sh.x_col);
-                g[i] = load_vec<VEC>(row + sh.g_col);
             } else {
 #pragma unroll
-                for (int j = 0; j < VEC; ++j) a[i].v[j] = b[i].v[j] = g[i].v[j] = 0.0f;
+                for (int j = 0; j < VEC; ++j) a[i].v[j] = b[i].v[j] = 0.0f;
             }
         }
         Pack<VEC> A, B;                       // this warp's stretch
@@ -169,7 +175,7 @@ gated_average_walk_kernel(const Shape sh, TO* __restrict__ out) {
 #pragma unroll
             for (int j = 0; j < VEC; ++j) {
                 float keep = 1.0f, add = 0.0f;
-                if (on) gates(a[i].v[j] + zb.v[j], b[i].v[j] + xb.v[j], keep, add);
+                if (on) gates<quick<TO>()>(a[i].v[j] + zb.v[j], b[i].v[j] + xb.v[j], keep, add);
                 a[i].v[j] = keep;
                 b[i].v[j] = add;
                 A.v[j] *= keep;
@@ -201,6 +207,21 @@ gated_average_walk_kernel(const Shape sh, TO* __restrict__ out) {
             store_vec<VEC>(&cta_a[parity][lane * VEC], CA);
             store_vec<VEC>(&cta_b[parity][lane * VEC], CB);
         }
+        // the first half's output gates are on their way while the cluster meets
+        Pack<VEC> g[TOKENS / 2];
+        auto load_gates = [&](int half) {
+#pragma unroll
+            for (int i = 0; i < TOKENS / 2; ++i) {
+                const int t = t0 + half * (TOKENS / 2) + i;
+                if (live && t < last) {
+                    g[i] = load_vec<VEC>(sh.p + (size_t)t * sh.row_stride + c + sh.g_col);
+                } else {
+#pragma unroll
+                    for (int j = 0; j < VEC; ++j) g[i].v[j] = 0.0f;
+                }
+            }
+        };
+        load_gates(0);
         cluster.sync();
         // the state in front of this CTA's stretch, and the one behind the round
         Pack<VEC> front = s;
@@ -215,11 +236,12 @@ gated_average_walk_kernel(const Shape sh, TO* __restrict__ out) {
         for (int j = 0; j < VEC; ++j) front.v[j] = fmaf(PA.v[j], front.v[j], PB.v[j]);
 #pragma unroll
         for (int i = 0; i < TOKENS; ++i) {
+            if (i == TOKENS / 2) load_gates(1);
             Pack<VEC> y;
 #pragma unroll
             for (int j = 0; j < VEC; ++j) {
                 front.v[j] = fmaf(a[i].v[j], front.v[j], b[i].v[j]);
-                y.v[j] = live ? front.v[j] * silu_f32(g[i].v[j]) : 0.0f;
+                y.v[j] = live ? front.v[j] * gate_out<quick<TO>()>(g[i % (TOKENS / 2)].v[j]) : 0.0f;
             }
             if (t0 + i < last && c < sh.ld_out) store_vec<VEC>(out + (size_t)(t0 + i) * sh.ld_out + c, y);
         }
@@ -260,10 +282,8 @@ int run(const Shape& sh, TO* out, int segments, int max_segment, int vec, cudaSt
     }
     int ranks = 1;
     while (ranks < 8 && ranks * STRETCH < max_segment) ranks *= 2;
-    // four channels a lane when that still gives the GPU a CTA or so for every SM
-    if (vec == 4 && (long)ranks * ((sh.ld_out + 127) / 128) * segments < 120) vec = 2;
-    if (vec == 4) return launch_walk<4, TO>(sh, out, segments, ranks, stream);
-    if (vec == 2) return launch_walk<2, TO>(sh, out, segments, ranks, stream);
+    // (two channels a lane: with four, a warp's eight tokens do not fit the registers of two CTAs an SM)
+    if (vec >= 2) return launch_walk<2, TO>(sh, out, segments, ranks, stream);
     return launch_walk<1, TO>(sh, out, segments, ranks, stream);
 }
 

@@ -7,6 +7,8 @@
     python -m flyweight_b200.kernels.microbench shortconv --tokens 2048
     python -m flyweight_b200.kernels.microbench qk-norm-rope --tokens 2048
     python -m flyweight_b200.kernels.microbench causal-conv --tokens 16384
+    python -m flyweight_b200.kernels.microbench gated-average --tokens 2048
+    python -m flyweight_b200.kernels.microbench route --tokens 2048
     python -m flyweight_b200.kernels.microbench sample --rows 8 --top-k 40
 
 It is what the ncu summaries under ``profiles/`` were captured from (small cases of the same
@@ -144,9 +146,13 @@ def run_attention_prefill(args) -> dict:
     tile_seg = torch.zeros(n_tiles, dtype=torch.int32, device="cuda")
     tile_tok0 = (torch.arange(n_tiles, dtype=torch.int32) * per_tile).cuda()
     scale = 1.0 / math.sqrt(args.head_dim)
+    if args.softcap:
+        extra["softcap"] = args.softcap
+    if args.keep_first:
+        extra["keep_first"] = args.keep_first
     kernel = ops.attention_prefill_mma if args.mma_sync else ops.attention_prefill_tcgen05
     us = _time(lambda: kernel(q, k_pool, v_pool, positions, seg_start, tile_seg, tile_tok0, n_tiles,
-                              per_tile, table, args.heads, 0, scale, **extra), args.repeat)
+                              per_tile, table, args.heads, args.window, scale, **extra), args.repeat)
     flops = 2.0 * T * T * args.heads * args.head_dim        # causal: half of 4*T*T*h*d
     from . import tensorcore
     return {"kernel": "attention_prefill_mma" if args.mma_sync else "attention_prefill_tcgen05",
@@ -253,6 +259,41 @@ def run_linear_attention(args) -> dict:
             "gflops": 4.0 * T * H * d * e / us / 1e3}
 
 
+def run_gated_average(args) -> dict:
+    """The minGRU recurrence over ``batch`` segments of ``tokens`` tokens, ``width`` channels.  The projections
+    are rotated through enough copies to exceed L2."""
+    from ..engine.batch import Segment, StepBatch
+    from . import mixing
+    W, T = args.width, args.batch * args.tokens
+    dev = torch.device("cuda", 0)
+    dtype = torch.float32 if args.fp32 else torch.bfloat16
+    row_bytes = T * 3 * W * 4
+    copies = [torch.randn((T, 3 * W), device=dev) for _ in range(max(1, -(-(256 << 20) // row_bytes)))]
+    bias = torch.zeros(W, device=dev)
+    state = torch.zeros((args.batch, W), device=dev)
+    batch = StepBatch([Segment(f"r{i}", i, 0, [0] * args.tokens, []) for i in range(args.batch)],
+                      [[[0]] * args.batch], dev)
+
+    def steps():
+        for p in copies:
+            mixing.gated_average(p, 0, W, 2 * W, bias, bias, state, batch, W, dtype)
+
+    us = _time_graph(steps, args.repeat) / len(copies)
+    moved = row_bytes + T * W * (4 if args.fp32 else 2) + 2 * args.batch * W * 4
+    return {"kernel": "gated_average", "batch": args.batch, "tokens": args.tokens, "width": W, "us": us,
+            "gb_s": moved / us / 1e3}
+
+
+def run_route(args) -> dict:
+    """The router of routed experts: scores of ``outputs`` outputs and the choice of ``top``."""
+    from . import experts
+    h = torch.randn((args.tokens, args.hidden), device="cuda").to(torch.bfloat16)
+    router = torch.randn((args.outputs, args.hidden), device="cuda") / math.sqrt(args.hidden)
+    us = _time_graph(lambda: experts.route(h, router, None, 1, 1, args.top, args.scores), args.repeat)
+    return {"kernel": "moe_route", "tokens": args.tokens, "outputs": args.outputs, "top": args.top, "us": us,
+            "gflops": 2.0 * args.tokens * args.outputs * args.hidden / us / 1e3}
+
+
 def run_qk_norm_rope(args) -> dict:
     from . import ops
     T, nh, nkv, hd = args.tokens, args.heads, args.kv_heads, args.head_dim
@@ -347,6 +388,9 @@ def main(argv=None) -> int:
                        help="one pool head for all query heads, rows as keys and values, a sink per head")
         p.add_argument("--graph", action="store_true",
                        help="decode: the launches captured in a CUDA graph (kernels shorter than a Python call)")
+        p.add_argument("--window", type=int, default=0, help="prefill: a sliding window")
+        p.add_argument("--keep-first", type=int, default=0, help="prefill: positions kept beside the window")
+        p.add_argument("--softcap", type=float, default=0.0)
         p.add_argument("--mma-sync", action="store_true", help="the mma.sync prompt kernel")
         p.add_argument("--cluster-merge", action="store_true", help="with --splits <= 8: merge inside the kernel")
         p.add_argument("--cp-async", action="store_true", help="decode: key and value tiles by cp.async, not TMA")
@@ -384,6 +428,17 @@ def main(argv=None) -> int:
     lin.add_argument("--dim", type=int, default=128)
     lin.add_argument("--vdim", type=int, default=128)
     lin.add_argument("--scan", action="store_true", help="the token-by-token kernel")
+    avg = sub.add_parser("gated-average")
+    avg.add_argument("--batch", type=int, default=1)
+    avg.add_argument("--tokens", type=int, default=2048)
+    avg.add_argument("--width", type=int, default=2048)
+    avg.add_argument("--fp32", action="store_true")
+    rt = sub.add_parser("route")
+    rt.add_argument("--tokens", type=int, default=2048)
+    rt.add_argument("--hidden", type=int, default=2048)
+    rt.add_argument("--outputs", type=int, default=32)
+    rt.add_argument("--top", type=int, default=8)
+    rt.add_argument("--scores", default="sigmoid")
     smp = sub.add_parser("sample")
     smp.add_argument("--rows", type=int, default=8)
     smp.add_argument("--vocab", type=int, default=65536)
@@ -399,7 +454,7 @@ def main(argv=None) -> int:
               "attention-prefill": run_attention_prefill, "shortconv": run_shortconv,
               "causal-conv": run_causal_conv,
               "qk-norm-rope": run_qk_norm_rope, "sample": run_sample, "delta-rule": run_delta_rule,
-              "linear-attention": run_linear_attention}[args.kernel]
+              "linear-attention": run_linear_attention, "gated-average": run_gated_average, "route": run_route}[args.kernel]
     print(json.dumps(runner(args)))
     return 0
 

@@ -394,5 +394,84 @@ FOBATAR_E = {
 TINY.update({"FA": FOBATAR_A, "FB": FOBATAR_B, "FC": FOBATAR_C, "FD": FOBATAR_D, "FE": FOBATAR_E})
 
 
+def _mingru(width):
+    return {"type": "mingru", "mixer": {"width": width}}
+
+
+def _parallel(left, right, left_scale, right_scale):
+    heads, kv_heads, dim, vdim, scale, more = left
+    r_heads, r_dim, r_vdim = right
+    decay = [round(1.0 - 0.3 / 2.0 ** (2 * h + 0.5), 6) for h in range(r_heads)]
+    return {"type": "parallel", "mixer": {
+        "left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, **more},
+        "right": {"heads": r_heads, "dim": r_dim, "vdim": r_vdim, "decay": decay},
+        "left_scale": left_scale, "right_scale": right_scale}}
+
+
+def _sigmoid_experts(ff, experts, top):
+    return {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+
+
+def _kept_window(size, keep_first, base=None, dims=0, softcap=None):
+    more = {"mask": {"size": size, "keep_first": keep_first}}
+    if base is not None:
+        more["rot"] = {"base": base, "dims": dims}
+    if softcap is not None:
+        more["softcap"] = softcap
+    return more
+
+
+# Tiny Vugipel configurations that differ in every size and option: windows shorter than, equal to and longer than
+# a page (and of one key), 0 to 70 kept first tokens (inside a page, a whole page, across a border), keys and
+# values of equal and of different sizes both ways, sizes that are no multiple of 16 or 8, rotation of all, some
+# and no key channels (values turn all the same) and no rotation, 1 to 4 query heads per key head, caps that
+# act and none, minGRU widths that are odd, even and larger than the model, equal and different pair scales (one
+# negative), one to all experts per token, layers without a feed-forward, models of one mixer only.
+VUGIPEL_A = {
+    "architecture": "Vugipel", "vocab": 211, "width": 80, "norm": {"eps": 1e-5},
+    "layers": [
+        {**_parallel((4, 2, 16, 24, 0.6, _kept_window(37, 5, 10000.0, 8, 2.0)), (3, 12, 20), 0.6, 1.1), "mlp": _sigmoid_experts(48, 5, 2)},
+        {**_mingru(52), "mlp": _sigmoid_experts(32, 3, 1)},
+        {**_mingru(100), "mlp": None},
+        {**_parallel((2, 1, 24, 24, 0.4, _kept_window(64, 64, 500.0, 24)), (1, 20, 8), 1.0, 1.0), "mlp": _sigmoid_experts(16, 4, 4)},
+    ],
+}
+VUGIPEL_B = {
+    "architecture": "Vugipel", "vocab": 130, "width": 96, "norm": {"eps": 1e-6},
+    "layers": [
+        {**_mingru(33), "mlp": _sigmoid_experts(24, 2, 2)},
+        {**_parallel((3, 3, 20, 12, 0.5, _kept_window(5, 1, 300.0, 0, 8.0)), (2, 33, 7), -0.5, 0.9), "mlp": None},
+        {**_parallel((6, 2, 8, 16, 0.7, {}), (4, 16, 16), 0.8, 0.3), "mlp": _sigmoid_experts(40, 7, 3)},
+        {**_mingru(18), "mlp": _sigmoid_experts(24, 2, 1)},
+    ],
+}
+# Sizes that the tensor-core kernels take, so that the bfloat16 path runs them: heads of 64 and 128 channels, four
+# query heads per key head, expert widths in multiples of 8.
+VUGIPEL_C = {
+    "architecture": "Vugipel", "vocab": 300, "width": 128, "norm": {"eps": 1e-5},
+    "layers": [
+        {**_mingru(128), "mlp": _sigmoid_experts(64, 6, 2)},
+        {**_parallel((8, 2, 64, 64, 0.2, _kept_window(130, 70, 1000000.0, 32, 4.0)), (2, 64, 64), 0.9, 0.7), "mlp": _sigmoid_experts(32, 4, 3)},
+        {**_parallel((4, 1, 128, 128, 0.15, _kept_window(70, 3, 10000.0, 128)), (4, 32, 48), 0.75, 1.25), "mlp": _sigmoid_experts(64, 6, 2)},
+        {**_mingru(192), "mlp": _sigmoid_experts(128, 3, 2)},
+    ],
+}
+# One mixer only.
+VUGIPEL_D = {
+    "architecture": "Vugipel", "vocab": 97, "width": 48, "norm": {"eps": 1e-6},
+    "layers": [{**_mingru(64), "mlp": _sigmoid_experts(80, 3, 2)}, {**_mingru(21), "mlp": None}, {**_mingru(64), "mlp": _sigmoid_experts(8, 1, 1)}],
+}
+VUGIPEL_E = {
+    "architecture": "Vugipel", "vocab": 160, "width": 64, "norm": {"eps": 1e-5},
+    "layers": [
+        {**_parallel((4, 2, 16, 32, 0.6, _kept_window(1, 3, 10000.0, 16)), (2, 24, 16), 1.3, 0.6), "mlp": _sigmoid_experts(96, 8, 1)},
+        {**_parallel((2, 2, 32, 16, 0.4, _kept_window(33, 0, 1000.0, 20, 3.0)), (5, 8, 24), 0.5, 0.5), "mlp": _sigmoid_experts(64, 2, 1)},
+        {**_parallel((2, 2, 32, 16, 0.4, _kept_window(100, 40)), (1, 64, 40), 0.5, 0.9), "mlp": _sigmoid_experts(64, 4, 2)},
+    ],
+}
+
+TINY.update({"VA": VUGIPEL_A, "VB": VUGIPEL_B, "VC": VUGIPEL_C, "VD": VUGIPEL_D, "VE": VUGIPEL_E})
+
+
 def vocab_of(config: dict) -> int:
     return int(config.get("vocab_size", config.get("vocab")))
