@@ -174,14 +174,36 @@ __device__ __forceinline__ void softmax_update(float (&s)[NT][4], float (&o)[HD 
     // capped scores: cap * tanh(score / cap), in base 2 like the scale (which has log2(e) folded in)
     const float cap_pre = softcap > 0.0f ? scale / (softcap * LOG2E) : 0.0f, cap_post = softcap * LOG2E;
     float mx[2] = {-INFINITY, -INFINITY};
+    if (softcap > 0.0f) {
+        // far below the cap (a whole warp's scores of this tile) the polynomial does; it spares the special-function
+        // unit, which the exponentials need
+        float top = 0.0f;
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                s[n][j] *= cap_pre;
+                top = fmaxf(top, fabsf(s[n][j]));
+            }
+        const bool small = __all_sync(0xffffffffu, top <= fwb::TANH_SMALL);
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                s[n][j] = cap_post * (small ? fwb::tanh_small_f32(s[n][j]) : fwb::tanh_fast_f32(s[n][j]));
+    } else {
+#pragma unroll
+        for (int n = 0; n < NT; ++n)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) s[n][j] *= scale;                  // scale has log2(e) folded in
+    }
 #pragma unroll
     for (int n = 0; n < NT; ++n)
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
             const int key = key_base + n * 8 + 2 * t + (j & 1);
             const int h = j >> 1;
-            const float capped = softcap > 0.0f ? cap_post * fwb::tanh_fast_f32(s[n][j] * cap_pre) : s[n][j] * scale;
-            const float v = ((key >= lo[h] || key < keep) && key <= hi[h]) ? capped : -INFINITY;   // scale has log2(e) folded in
+            const float v = ((key >= lo[h] || key < keep) && key <= hi[h]) ? s[n][j] : -INFINITY;
             s[n][j] = v;
             mx[h] = fmaxf(mx[h], v);
         }

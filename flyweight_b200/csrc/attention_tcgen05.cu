@@ -335,8 +335,21 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
                 tmem_ld64(lane_addr + buf * KEYS, sc);
                 tc_fence_before();                         // S is out of its buffer before this warp says that P is ready
                 if (prm.cap_pre != 0.0f) {
+                    // a warp whose scores of this tile all lie far below the cap takes the polynomial: it spares the
+                    // special-function unit, which the exponentials need
+                    float top = 0.0f;
 #pragma unroll
-                    for (int i = 0; i < KEYS; ++i) sc[i] = prm.cap_unit * fwb::tanh_fast_f32(sc[i] * prm.cap_pre);
+                    for (int i = 0; i < KEYS; ++i) {
+                        sc[i] *= prm.cap_pre;
+                        top = fmaxf(top, fabsf(sc[i]));
+                    }
+                    if (__all_sync(0xffffffffu, top <= fwb::TANH_SMALL)) {
+#pragma unroll
+                        for (int i = 0; i < KEYS; ++i) sc[i] = prm.cap_unit * fwb::tanh_small_f32(sc[i]);
+                    } else {
+#pragma unroll
+                        for (int i = 0; i < KEYS; ++i) sc[i] = prm.cap_unit * fwb::tanh_fast_f32(sc[i]);
+                    }
                 }
                 // a tile every row sees whole needs no mask (rows without a token are never stored)
                 const bool whole = (key0 >= lo_max || key0 + KEYS <= prm.keep) && key0 + KEYS - 1 <= item.pos_first;

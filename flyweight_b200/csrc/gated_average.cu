@@ -135,6 +135,7 @@ gated_average_walk_kernel(const Shape sh, TO* __restrict__ out) {
     constexpr int COLS = 32 * VEC;
     __shared__ __align__(16) float warp_a[WARPS][COLS], warp_b[WARPS][COLS];
     __shared__ __align__(16) float cta_a[2][COLS], cta_b[2][COLS];          // this CTA's stretch, by round parity
+    __shared__ __align__(16) float all_a[8][COLS], all_b[8][COLS];          // every CTA's stretch of the round
     cg::cluster_group cluster = cg::this_cluster();
     const int ranks = gridDim.x, rank = blockIdx.x;                          // the cluster spans the grid's x
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -189,6 +190,7 @@ gated_average_walk_kernel(const Shape sh, TO* __restrict__ out) {
         Pack<VEC> PA, PB;
 #pragma unroll
         for (int j = 0; j < VEC; ++j) PA.v[j] = 1.0f, PB.v[j] = 0.0f;
+#pragma unroll 5
         for (int w = 0; w < warp; ++w) {
             const Pack<VEC> wa = load_vec<VEC>(&warp_a[w][lane * VEC]), wb = load_vec<VEC>(&warp_b[w][lane * VEC]);
 #pragma unroll
@@ -223,12 +225,18 @@ gated_average_walk_kernel(const Shape sh, TO* __restrict__ out) {
         };
         load_gates(0);
         cluster.sync();
+        // one warp fetches one CTA's stretch: a single trip through distributed shared memory
+        if (warp < ranks) {
+            store_vec<VEC>(&all_a[warp][lane * VEC], load_vec<VEC>(cluster.map_shared_rank(&cta_a[parity][lane * VEC], warp)));
+            store_vec<VEC>(&all_b[warp][lane * VEC], load_vec<VEC>(cluster.map_shared_rank(&cta_b[parity][lane * VEC], warp)));
+        }
+        __syncthreads();
         // the state in front of this CTA's stretch, and the one behind the round
         Pack<VEC> front = s;
+#pragma unroll 4
         for (int r = 0; r < ranks; ++r) {
             if (r == rank) front = s;
-            const Pack<VEC> ra = load_vec<VEC>(cluster.map_shared_rank(&cta_a[parity][lane * VEC], r));
-            const Pack<VEC> rb = load_vec<VEC>(cluster.map_shared_rank(&cta_b[parity][lane * VEC], r));
+            const Pack<VEC> ra = load_vec<VEC>(&all_a[r][lane * VEC]), rb = load_vec<VEC>(&all_b[r][lane * VEC]);
 #pragma unroll
             for (int j = 0; j < VEC; ++j) s.v[j] = fmaf(ra.v[j], s.v[j], rb.v[j]);
         }
@@ -246,7 +254,7 @@ gated_average_walk_kernel(const Shape sh, TO* __restrict__ out) {
             if (t0 + i < last && c < sh.ld_out) store_vec<VEC>(out + (size_t)(t0 + i) * sh.ld_out + c, y);
         }
         // (the next round writes warp_a / warp_b behind this round's cluster barrier, which every warp reached
-        // after reading them, and the other parity's cta_a / cta_b)
+        // after reading them, the other parity's cta_a / cta_b, and all_a / all_b behind its own barriers)
     }
     cluster.sync();                            // nobody leaves while a peer may still read its stretch
     if (rank == 0 && warp == 0 && live) store_vec<VEC>(mine, s);

@@ -31,6 +31,87 @@ namespace {
 constexpr int TM = 64, TN = 64, TK = 16;       // tile of the experts' products
 constexpr int SCORE_SIGMOID = 1;               // a router's scores: 0 softmax over the outputs, 1 sigmoid of each
 
+// One warp: from a token's router outputs s[N] (shared memory) to its scores, the choice inside the kept runs,
+// and the `top` chosen outputs with their scores.  choice[N], best[n_groups]: scratch in shared memory.
+__device__ __forceinline__ void choose_outputs(float* s, float* choice, float* best, const float* __restrict__ correction,
+                                               int* __restrict__ ids, float* __restrict__ weights, int N, int n_groups,
+                                               int keep, int top, int scoring) {
+    const int lane = threadIdx.x & 31;
+    if (scoring == SCORE_SIGMOID) {
+        for (int n = lane; n < N; n += 32) {
+            const float z = s[n], e = expf(-fabsf(z));
+            s[n] = z >= 0.0f ? 1.0f / (1.0f + e) : e / (1.0f + e);
+        }
+    } else {
+        float m = -INFINITY;
+        for (int n = lane; n < N; n += 32) m = fmaxf(m, s[n]);
+        m = warp_max(m);
+        float sum = 0.0f;
+        for (int n = lane; n < N; n += 32) sum += expf(s[n] - m);
+        sum = warp_sum(sum);
+        for (int n = lane; n < N; n += 32) s[n] = expf(s[n] - m) / sum;
+    }
+    for (int n = lane; n < N; n += 32) choice[n] = s[n] + (correction ? correction[n] : 0.0f);
+    __syncwarp();
+    const int per = N / n_groups;
+    for (int g = lane; g < n_groups; g += 32) {
+        float v = -INFINITY;
+        for (int j = 0; j < per; ++j) v = fmaxf(v, choice[g * per + j]);
+        best[g] = v;
+    }
+    __syncwarp();
+    // the (n_groups - keep) weakest runs leave the race, weakest first; ties: the higher index leaves
+    for (int out = 0; out < n_groups - keep; ++out) {
+        float v = INFINITY;
+        int at = -1;
+        for (int g = lane; g < n_groups; g += 32)
+            if (best[g] != INFINITY && (best[g] < v || (best[g] == v && g > at))) {
+                v = best[g];
+                at = g;
+            }
+        for (int offset = 16; offset > 0; offset >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, v, offset);
+            const int oat = __shfl_xor_sync(0xffffffffu, at, offset);
+            if (oat >= 0 && (at < 0 || ov < v || (ov == v && oat > at))) {
+                v = ov;
+                at = oat;
+            }
+        }
+        if (at < 0) break;
+        __syncwarp();
+        if (lane == 0) best[at] = INFINITY;        // marks a run that is out
+        for (int j = lane; j < per; j += 32) choice[at * per + j] = -INFINITY;
+        __syncwarp();
+    }
+    // the `top` largest choice values, largest first; ties: the lower index
+    for (int slot = 0; slot < top; ++slot) {
+        float v = -INFINITY;
+        int at = -1;
+        for (int n = lane; n < N; n += 32)
+            if (choice[n] > v || at < 0) {
+                if (choice[n] > v || at < 0) {
+                    v = choice[n];
+                    at = n;
+                }
+            }
+        for (int offset = 16; offset > 0; offset >>= 1) {
+            const float ov = __shfl_xor_sync(0xffffffffu, v, offset);
+            const int oat = __shfl_xor_sync(0xffffffffu, at, offset);
+            if (oat >= 0 && (at < 0 || ov > v || (ov == v && oat < at))) {
+                v = ov;
+                at = oat;
+            }
+        }
+        __syncwarp();
+        if (lane == 0) {
+            ids[slot] = at;
+            weights[slot] = s[at];
+            choice[at] = -INFINITY;
+        }
+        __syncwarp();
+    }
+}
+
 template <typename TH>
 __global__ void __launch_bounds__(512)
 moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, const float* __restrict__ correction,
@@ -125,79 +206,23 @@ moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, con
     }
     __syncthreads();
     if (warp != 0) return;
-    if (scoring == SCORE_SIGMOID) {
-        for (int n = lane; n < N; n += 32) {
-            const float z = s[n], e = expf(-fabsf(z));
-            s[n] = z >= 0.0f ? 1.0f / (1.0f + e) : e / (1.0f + e);
-        }
-    } else {
-        float m = -INFINITY;
-        for (int n = lane; n < N; n += 32) m = fmaxf(m, s[n]);
-        m = warp_max(m);
-        float sum = 0.0f;
-        for (int n = lane; n < N; n += 32) sum += expf(s[n] - m);
-        sum = warp_sum(sum);
-        for (int n = lane; n < N; n += 32) s[n] = expf(s[n] - m) / sum;
-    }
-    for (int n = lane; n < N; n += 32) choice[n] = s[n] + (correction ? correction[n] : 0.0f);
+    choose_outputs(s, choice, best, correction, ids + (size_t)t * top, weights + (size_t)t * top, N, n_groups, keep, top, scoring);
+}
+
+// The choice alone, from router outputs that a matrix product made: one warp a token.
+__global__ void __launch_bounds__(128)
+moe_choose_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int* __restrict__ ids,
+                  float* __restrict__ weights, int T, int N, int n_groups, int keep, int top, int scoring) {
+    fwb::pdl_entry();
+    extern __shared__ float shared[];
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int t = blockIdx.x * (blockDim.x >> 5) + warp;
+    if (t >= T) return;
+    float* s = shared + warp * (2 * N + n_groups);
+    for (int n = lane; n < N; n += 32) s[n] = logits[(size_t)t * N + n];
     __syncwarp();
-    const int per = N / n_groups;
-    for (int g = lane; g < n_groups; g += 32) {
-        float v = -INFINITY;
-        for (int j = 0; j < per; ++j) v = fmaxf(v, choice[g * per + j]);
-        best[g] = v;
-    }
-    __syncwarp();
-    // the (n_groups - keep) weakest runs leave the race, weakest first; ties: the higher index leaves
-    for (int out = 0; out < n_groups - keep; ++out) {
-        float v = INFINITY;
-        int at = -1;
-        for (int g = lane; g < n_groups; g += 32)
-            if (best[g] != INFINITY && (best[g] < v || (best[g] == v && g > at))) {
-                v = best[g];
-                at = g;
-            }
-        for (int offset = 16; offset > 0; offset >>= 1) {
-            const float ov = __shfl_xor_sync(0xffffffffu, v, offset);
-            const int oat = __shfl_xor_sync(0xffffffffu, at, offset);
-            if (oat >= 0 && (at < 0 || ov < v || (ov == v && oat > at))) {
-                v = ov;
-                at = oat;
-            }
-        }
-        if (at < 0) break;
-        __syncwarp();
-        if (lane == 0) best[at] = INFINITY;        // marks a run that is out
-        for (int j = lane; j < per; j += 32) choice[at * per + j] = -INFINITY;
-        __syncwarp();
-    }
-    // the `top` largest choice values, largest first; ties: the lower index
-    for (int slot = 0; slot < top; ++slot) {
-        float v = -INFINITY;
-        int at = -1;
-        for (int n = lane; n < N; n += 32)
-            if (choice[n] > v || at < 0) {
-                if (choice[n] > v || at < 0) {
-                    v = choice[n];
-                    at = n;
-                }
-            }
-        for (int offset = 16; offset > 0; offset >>= 1) {
-            const float ov = __shfl_xor_sync(0xffffffffu, v, offset);
-            const int oat = __shfl_xor_sync(0xffffffffu, at, offset);
-            if (oat >= 0 && (at < 0 || ov > v || (ov == v && oat < at))) {
-                v = ov;
-                at = oat;
-            }
-        }
-        __syncwarp();
-        if (lane == 0) {
-            ids[(size_t)t * top + slot] = at;
-            weights[(size_t)t * top + slot] = s[at];
-            choice[at] = -INFINITY;
-        }
-        __syncwarp();
-    }
+    choose_outputs(s, s + N, s + 2 * N, correction, ids + (size_t)t * top, weights + (size_t)t * top, N, n_groups, keep, top,
+                   scoring);
 }
 
 // A router that is a table: token id -> its `top` experts, each with weight 1 / top.
@@ -226,37 +251,66 @@ moe_sort_kernel(const int* __restrict__ ids, int A, int top, int E, int tile_row
                 int* __restrict__ row_token, int* __restrict__ pair_row, int* __restrict__ tiles,
                 const float* __restrict__ weights, float* __restrict__ row_weight) {
     fwb::pdl_entry();
+    // Lanes of a warp that hold the same expert add once for all of them (a step of thousands of pairs over a few
+    // dozen experts would otherwise queue on every counter).
     extern __shared__ int counts[];               // [E] counts, then [E] cursors
     int* cursor = counts + E;
+    const int lane = threadIdx.x & 31;
     for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
     __syncthreads();
-    for (int a = threadIdx.x; a < A; a += blockDim.x) {
-        const int e = ids[a];
-        if (e >= 0 && e < E) atomicAdd(&counts[e], 1);
+    const int turns = (A + blockDim.x - 1) / blockDim.x;
+    for (int turn = 0; turn < turns; ++turn) {
+        const int a = turn * blockDim.x + threadIdx.x;
+        const int e = a < A ? ids[a] : -1;
+        const unsigned same = __match_any_sync(0xffffffffu, e);
+        if (e >= 0 && e < E && lane == __ffs(same) - 1) atomicAdd(&counts[e], __popc(same));
     }
     __syncthreads();
-    if (threadIdx.x == 0) {
-        int at = 0, n_tiles = 0;
-        for (int e = 0; e < E; ++e) {
-            const int n = counts[e];
-            offsets[e] = at;
-            cursor[e] = at;
-            for (int row = 0; row < n; row += tile_rows) {
-                tiles[1 + 2 * n_tiles] = e;
-                tiles[2 + 2 * n_tiles] = at + row;
-                ++n_tiles;
+    if (threadIdx.x < 32) {
+        // first rows and first tiles of the experts, 32 experts at a time
+        int row0 = 0, tile0 = 0;
+        for (int e0 = 0; e0 < E; e0 += 32) {
+            const int e = e0 + lane, n = e < E ? counts[e] : 0, t = (n + tile_rows - 1) / tile_rows;
+            int rows = n, tile_end = t;
+#pragma unroll
+            for (int step = 1; step < 32; step <<= 1) {
+                const int r = __shfl_up_sync(0xffffffffu, rows, step), u = __shfl_up_sync(0xffffffffu, tile_end, step);
+                if (lane >= step) {
+                    rows += r;
+                    tile_end += u;
+                }
             }
-            at += n;
+            if (e < E) {
+                const int at = row0 + rows - n, first = tile0 + tile_end - t;
+                offsets[e] = at;
+                cursor[e] = at;
+                for (int i = 0; i < t; ++i) {
+                    tiles[1 + 2 * (first + i)] = e;
+                    tiles[2 + 2 * (first + i)] = at + i * tile_rows;
+                }
+            }
+            row0 += __shfl_sync(0xffffffffu, rows, 31);
+            tile0 += __shfl_sync(0xffffffffu, tile_end, 31);
         }
-        offsets[E] = at;
-        tiles[0] = n_tiles;
+        if (lane == 0) {
+            offsets[E] = row0;
+            tiles[0] = tile0;
+        }
     }
     __syncthreads();
-    for (int a = threadIdx.x; a < A; a += blockDim.x) {
-        const int e = ids[a];
+    for (int turn = 0; turn < turns; ++turn) {
+        const int a = turn * blockDim.x + threadIdx.x;
+        const int e = a < A ? ids[a] : -1;
+        const bool real = e >= 0 && e < E;
+        const unsigned same = __match_any_sync(0xffffffffu, e);
+        const int leader = __ffs(same) - 1;
+        int base = 0;
+        if (real && lane == leader) base = atomicAdd(&cursor[e], __popc(same));
+        base = __shfl_sync(0xffffffffu, base, leader);
+        if (a >= A) continue;
         int row = -1;
-        if (e >= 0 && e < E) {
-            row = atomicAdd(&cursor[e], 1);
+        if (real) {
+            row = base + __popc(same & ((1u << lane) - 1));
             row_token[row] = a / top;
             if (row_weight) row_weight[row] = weights[a];
         }
@@ -534,6 +588,20 @@ FWB_API int fwb_moe_route(const void* h, int h_bf16, const float* router, const 
     else
         fwb::pdl(moe_route_kernel<float>, blocks, threads, smem, stream)((const float*)h, router, correction, ids,
                                                                           weights, T, W, N, n_groups, keep, top, vec, scoring);
+    return fwb_launch_status();
+}
+
+// The same choice from router outputs that are there already: logits fp32 [T][N].
+FWB_API int fwb_moe_choose(const float* logits, const float* correction, int* ids, float* weights, int T, int N,
+                           int n_groups, int keep, int top, int scoring, cudaStream_t stream) {
+    if (T <= 0) return FWB_OK;
+    if (!logits || !ids || !weights || scoring < 0 || scoring > 1) return FWB_BAD_ARGUMENT;
+    if (N <= 0 || n_groups <= 0 || N % n_groups || keep <= 0 || keep > n_groups || top <= 0 || top > keep * (N / n_groups))
+        return FWB_BAD_ARGUMENT;
+    const size_t smem = (size_t)4 * (2 * N + n_groups) * sizeof(float);
+    if (smem > 48 * 1024) return FWB_TOO_LARGE;
+    fwb::pdl(moe_choose_kernel, (T + 3) / 4, 128, smem, stream)(logits, correction, ids, weights, T, N, n_groups, keep, top,
+                                                                scoring);
     return fwb_launch_status();
 }
 

@@ -21,14 +21,17 @@ def set_tensor_cores(flag: bool) -> None:
     _use_tensor_cores = bool(flag)
 
 
+TENSOR_CORE_ROUTER_FROM = 256      # tokens of a step from which a bfloat16 router is a matrix product
 ROUTER_SCORES = {"softmax": 0, "sigmoid": 1}
 
 
 def route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], n_groups: int, keep: int, top: int,
-          scores: str = "softmax"):
+          scores: str = "softmax", router16: Optional[torch.Tensor] = None):
     """ids int32 [T][top] and weights fp32 [T][top]: ``scores`` "softmax" over all router outputs or the
     "sigmoid" of each; the choice on score (+ correction) inside the ``keep`` best of ``n_groups`` runs of
-    neighbours; the weights are the chosen outputs' plain scores."""
+    neighbours; the weights are the chosen outputs' plain scores.  ``router16``: the same router in bfloat16, when
+    that loses nothing: bfloat16 rows of a prompt then take the tensor-core product (products of bfloat16 numbers
+    are exact in fp32, and so is what they are summed in) and a kernel that only chooses."""
     check_tensor("router input", h)
     T, W = h.shape
     N = router.shape[0]
@@ -39,6 +42,16 @@ def route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tens
         raise KernelError(f"unknown router scores {scores!r}; known: " + ", ".join(ROUTER_SCORES))
     ids = torch.empty((T, top), dtype=torch.int32, device=h.device)
     weights = torch.empty((T, top), dtype=torch.float32, device=h.device)
+    if router16 is not None and T >= TENSOR_CORE_ROUTER_FROM and h.dtype == torch.bfloat16:
+        from . import tensorcore
+        if tensorcore.accepts(h, router16, torch.float32):
+            # one tile of features: token tiles and slices of K make the CTAs
+            tile = 64 if T <= 2048 else 128
+            splits = 4 if -(-T // tile) <= 37 and W >= 1024 else (2 if -(-T // tile) <= 74 and W >= 512 else 1)
+            logits = tensorcore.gemm(h, router16, torch.float32, splits=splits, tile_tokens=tile)
+            lib.call("fwb_moe_choose", ptr(logits), ptr(correction), ptr(ids), ptr(weights), T, N, int(n_groups), int(keep),
+                     int(top), ROUTER_SCORES[scores], stream())
+            return ids, weights
     lib.call("fwb_moe_route", ptr(h), is_bf16(h), ptr(router), ptr(correction), ptr(ids), ptr(weights), T, W, N,
              int(n_groups), int(keep), int(top), ROUTER_SCORES[scores], stream())
     return ids, weights

@@ -289,7 +289,10 @@ def run_route(args) -> dict:
     from . import experts
     h = torch.randn((args.tokens, args.hidden), device="cuda").to(torch.bfloat16)
     router = torch.randn((args.outputs, args.hidden), device="cuda") / math.sqrt(args.hidden)
-    us = _time_graph(lambda: experts.route(h, router, None, 1, 1, args.top, args.scores), args.repeat)
+    router16 = router.to(torch.bfloat16)
+    router = router16.float()
+    us = _time_graph(lambda: experts.route(h, router, None, 1, 1, args.top, args.scores,
+                                           None if args.simt else router16), args.repeat)
     return {"kernel": "moe_route", "tokens": args.tokens, "outputs": args.outputs, "top": args.top, "us": us,
             "gflops": 2.0 * args.tokens * args.outputs * args.hidden / us / 1e3}
 
@@ -438,6 +441,7 @@ def main(argv=None) -> int:
     rt.add_argument("--hidden", type=int, default=2048)
     rt.add_argument("--outputs", type=int, default=32)
     rt.add_argument("--top", type=int, default=8)
+    rt.add_argument("--simt", action="store_true", help="the fp32-FMA kernel at every size")
     rt.add_argument("--scores", default="sigmoid")
     smp = sub.add_parser("sample")
     smp.add_argument("--rows", type=int, default=8)

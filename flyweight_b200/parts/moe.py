@@ -53,7 +53,7 @@ class RoutedExperts(FeedForward):
                              f"{self.keep_groups} are kept")
         if not 0 < self.top <= self.keep_groups * (outputs // self.groups):
             raise ValueError(f"top {self.top} does not fit the {self.keep_groups} kept groups")
-        self.router = self.correction = self.w_gate_up = self.w_down = None
+        self.router = self.router16 = self.correction = self.w_gate_up = self.w_down = None
 
     @property
     def n_outputs(self) -> int:
@@ -73,7 +73,10 @@ class RoutedExperts(FeedForward):
     def bind(self, get, precision: Precision, device):
         n = self.names
         # the router runs in fp32 whatever the precision (a bfloat16 matrix widens exactly)
-        self.router = precision.vector(get(n["router"]), device)
+        stored = get(n["router"])
+        self.router = precision.vector(stored, device)
+        # (stored in bfloat16: the same numbers, for the tensor-core product of a prompt's rows)
+        self.router16 = stored.to(device).contiguous() if stored.dtype == torch.bfloat16 and precision.name == "bfloat16" else None
         if self.corrected:
             self.correction = precision.vector(get(n["correction"]), device)
         mats = [get(n[f"{role}{j}"]) for j in range(self.n_experts) for role in ("gate", "up", "down")]
@@ -106,7 +109,7 @@ class RoutedExperts(FeedForward):
 
     def forward(self, ctx, h, add_normed_into=None):
         ids, weights = expert_kernels.route(h, self.router, self.correction, self.groups, self.keep_groups, self.top,
-                                            self.scores)
+                                            self.scores, self.router16)
         if h.dtype != self.w_gate_up.dtype:
             h = ops.cast(h, self.w_gate_up.dtype)
         return expert_kernels.experts_forward(h, ids, weights, self.w_gate_up, self.w_down, self.activation,
