@@ -246,24 +246,32 @@ moe_route_table_kernel(const int* __restrict__ token_ids, const int* __restrict_
 //   tiles[0]         number of row tiles (of tile_rows rows at most, none across two experts);
 //                    tiles[1 + 2 i], tiles[2 + 2 i]: expert and first row of tile i
 //   row_weight[A]    the pair's weight at its sorted row (only with `row_weight`)
+template <int HOLD>
 __global__ void __launch_bounds__(1024)
 moe_sort_kernel(const int* __restrict__ ids, int A, int top, int E, int tile_rows, int* __restrict__ offsets,
                 int* __restrict__ row_token, int* __restrict__ pair_row, int* __restrict__ tiles,
                 const float* __restrict__ weights, float* __restrict__ row_weight) {
     fwb::pdl_entry();
-    // Lanes of a warp that hold the same expert add once for all of them (a step of thousands of pairs over a few
-    // dozen experts would otherwise queue on every counter).
+    // A thread takes HOLD pairs at a time, their loads in flight together: one block walks all pairs, so what
+    // counts is how many round trips to memory lie one behind the other.
     extern __shared__ int counts[];               // [E] counts, then [E] cursors
     int* cursor = counts + E;
     const int lane = threadIdx.x & 31;
     for (int e = threadIdx.x; e < E; e += blockDim.x) counts[e] = 0;
     __syncthreads();
-    const int turns = (A + blockDim.x - 1) / blockDim.x;
-    for (int turn = 0; turn < turns; ++turn) {
-        const int a = turn * blockDim.x + threadIdx.x;
-        const int e = a < A ? ids[a] : -1;
-        const unsigned same = __match_any_sync(0xffffffffu, e);
-        if (e >= 0 && e < E && lane == __ffs(same) - 1) atomicAdd(&counts[e], __popc(same));
+    int held[HOLD];
+    auto take = [&](int a0) {
+#pragma unroll
+        for (int i = 0; i < HOLD; ++i) {
+            const int a = a0 + i * blockDim.x + threadIdx.x;
+            held[i] = a < A ? ids[a] : -1;
+        }
+    };
+    for (int a0 = 0; a0 < A; a0 += HOLD * blockDim.x) {
+        take(a0);
+#pragma unroll
+        for (int i = 0; i < HOLD; ++i)
+            if (held[i] >= 0 && held[i] < E) atomicAdd(&counts[held[i]], 1);
     }
     __syncthreads();
     if (threadIdx.x < 32) {
@@ -298,23 +306,21 @@ moe_sort_kernel(const int* __restrict__ ids, int A, int top, int E, int tile_row
         }
     }
     __syncthreads();
-    for (int turn = 0; turn < turns; ++turn) {
-        const int a = turn * blockDim.x + threadIdx.x;
-        const int e = a < A ? ids[a] : -1;
-        const bool real = e >= 0 && e < E;
-        const unsigned same = __match_any_sync(0xffffffffu, e);
-        const int leader = __ffs(same) - 1;
-        int base = 0;
-        if (real && lane == leader) base = atomicAdd(&cursor[e], __popc(same));
-        base = __shfl_sync(0xffffffffu, base, leader);
-        if (a >= A) continue;
-        int row = -1;
-        if (real) {
-            row = base + __popc(same & ((1u << lane) - 1));
-            row_token[row] = a / top;
-            if (row_weight) row_weight[row] = weights[a];
+    for (int a0 = 0; a0 < A; a0 += HOLD * blockDim.x) {
+        if (A > HOLD * blockDim.x) take(a0);           // (else the pairs are still held)
+        int rows[HOLD];
+#pragma unroll
+        for (int i = 0; i < HOLD; ++i)
+            rows[i] = held[i] >= 0 && held[i] < E ? atomicAdd(&cursor[held[i]], 1) : -1;
+#pragma unroll
+        for (int i = 0; i < HOLD; ++i) {
+            const int a = a0 + i * blockDim.x + threadIdx.x;
+            if (a >= A) continue;
+            pair_row[a] = rows[i];
+            if (rows[i] < 0) continue;
+            row_token[rows[i]] = a / top;
+            if (row_weight) row_weight[rows[i]] = weights[a];
         }
-        pair_row[a] = row;
     }
 }
 
@@ -624,7 +630,9 @@ FWB_API int fwb_moe_sort(const int* ids, int A, int top, int E, int tile_rows, i
         (weights == nullptr) != (row_weight == nullptr))
         return FWB_BAD_ARGUMENT;
     if (E > 4096) return FWB_TOO_LARGE;
-    fwb::pdl(moe_sort_kernel, 1, 1024, (size_t)(2 * E + 1) * sizeof(int), stream)(ids, A, top, E, tile_rows, offsets,
+    auto kernel = A <= 1024 ? moe_sort_kernel<1> : moe_sort_kernel<16>;
+    const int threads = A <= 128 ? 128 : (A <= 512 ? 512 : 1024);
+    fwb::pdl(kernel, 1, threads, (size_t)(2 * E + 1) * sizeof(int), stream)(ids, A, top, E, tile_rows, offsets,
                                                                                   row_token, pair_row, tiles, weights,
                                                                                   row_weight);
     return fwb_launch_status();

@@ -593,3 +593,51 @@ def test_experts_whose_inputs_are_weighted(dtype, tensor_cores, T, W, F, E, top)
     for on in want:
         close(got[on], want[on], 1e-5 if dtype == torch.float32 else 2e-2, on)
     assert (want["input"] - want["output"]).abs().max() > SHOWS * want["output"].abs().max()
+
+
+@pytest.mark.parametrize("T,W,N,top,groups,keep", [(256, 512, 32, 8, 1, 1), (700, 1024, 12, 3, 4, 2), (2049, 256, 5, 5, 1, 1), (300, 2048, 100, 1, 1, 1)])
+@pytest.mark.parametrize("scores", ["sigmoid", "softmax"])
+def test_the_router_as_a_matrix_product_chooses_alike(T, W, N, top, groups, keep, scores):
+    """bfloat16 rows of a prompt through the tensor-core product and the choosing kernel, against the kernel that does
+    both in fp32; where a choice is no close call it must be the same."""
+    from flyweight_b200.kernels import experts
+    g = torch.Generator().manual_seed(N)
+    h = torch.randn(T, W, generator=g).to(torch.bfloat16).to(DEV)
+    router16 = (2.0 * torch.randn(N, W, generator=g) / math.sqrt(W)).to(torch.bfloat16).to(DEV)
+    correction = (0.1 * torch.randn(N, generator=g)).to(DEV)
+    one = experts.route(h, router16.float(), correction, groups, keep, top, scores)
+    two = experts.route(h, router16.float(), correction, groups, keep, top, scores, router16=router16)
+    same = (one[0] == two[0]).all(dim=1)
+    assert same.float().mean() > 0.99
+    close(two[1][same], one[1][same], 1e-5)
+
+
+@pytest.mark.parametrize("A,top,E", [(1, 1, 1), (130, 2, 7), (1024, 4, 40), (1025, 5, 3), (17000, 4, 33), (40000, 8, 70)])
+@pytest.mark.parametrize("tile_rows", [16, 64])
+def test_pairs_are_sorted_by_expert(A, top, E, tile_rows):
+    """Every pair of a real expert gets one row among its expert's, the tiles cover the rows once and never two experts;
+    outputs from E on (identity experts) get no row."""
+    from flyweight_b200.kernels import lib
+    from flyweight_b200.kernels.lib import ptr, stream
+    g = torch.Generator().manual_seed(A)
+    ids = torch.randint(0, E + 1, (A,), generator=g).to(torch.int32)
+    weights = torch.rand(A, generator=g)
+    most = A // tile_rows + E + 1
+    offsets, row_token, pair_row, tiles = (torch.full((n,), -7, dtype=torch.int32, device=DEV) for n in (E + 1, A, A, 1 + 2 * most))
+    row_weight = torch.full((A,), -7.0, device=DEV)
+    ids_d, weights_d = dev(ids), dev(weights)
+    lib.call("fwb_moe_sort", ptr(ids_d), A, top, E, tile_rows, ptr(offsets), ptr(row_token), ptr(pair_row), ptr(tiles),
+             ptr(weights_d), ptr(row_weight), stream())
+    counts = torch.bincount(ids.long(), minlength=E + 1)[:E]
+    starts = torch.cat([torch.zeros(1, dtype=torch.long), counts.cumsum(0)])
+    assert offsets.cpu().long().tolist() == starts.tolist()
+    rows, total = pair_row.cpu().long(), int(starts[-1])
+    real = ids < E
+    assert (rows[~real] == -1).all() and sorted(rows[real].tolist()) == list(range(total))
+    expert_of_row = torch.repeat_interleave(torch.arange(E), counts)
+    assert (expert_of_row[rows[real]] == ids[real].long()).all()
+    pairs = torch.arange(A)[real]
+    assert (row_token.cpu().long()[rows[real]] == pairs // top).all() and (row_weight.cpu()[rows[real]] == weights[real]).all()
+    n = int(tiles[0])
+    listed = tiles[1:1 + 2 * n].cpu().view(n, 2).tolist()
+    assert listed == [[e, int(starts[e]) + r] for e in range(E) for r in range(0, int(counts[e]), tile_rows)] and n <= most
