@@ -1,9 +1,9 @@
 // A short causal convolution over time on every channel of a row buffer, with the rolling inputs of every
 // request kept between steps:
 //
-//     y[t][c] = sum_j taps[c][j] * u[t - n + 1 + j][c],   j = 0 .. n - 1,
+//     y[t][c] = act(bias[c] + sum_j taps[c][j] * u[t - n + 1 + j][c]),   j = 0 .. n - 1,
 //
-// where u before the start of a sequence is zero.  A step brings segments (runs of consecutive tokens of
+// where u before the start of a sequence is zero; the bias and act (silu) are optional.  A step brings segments (runs of consecutive tokens of
 // one request); the n - 1 inputs in front of a segment come from the request's state slot, which holds
 // the last n - 1 inputs of the sequence so far (oldest first, zero when the request starts).
 //
@@ -43,6 +43,16 @@ __device__ __forceinline__ float conv_one(const T* __restrict__ in, size_t at, l
     }
     return acc;
 }
+
+// What happens to a convolved value before it leaves: the channel's bias (null: none), then silu if asked for.
+struct ConvFinish {
+    const float* bias;
+    int silu;
+    __device__ __forceinline__ float operator()(float v, int c) const {
+        if (bias) v += bias[c];
+        return silu ? silu_f32(v) : v;
+    }
+};
 
 // Four consecutive channels of one row as fp32 (16 bytes of fp32, 8 of bfloat16).
 template <typename T> __device__ __forceinline__ float4 load4(const T* p);
@@ -89,12 +99,13 @@ __device__ __forceinline__ float2 block_sum2(float a, float b, float* scratch /*
 // convolved row stays in shared memory while the sums of squares of its one or two norm ranges are reduced,
 // then every entry leaves scaled (entries outside the ranges, or all of them when there is no range, leave as
 // they are).  C, ld, out_ld, col0 and the ranges' borders are multiples of four.
-template <typename T, int NT>
+template <typename T, typename TO, int NT>
 __global__ void __launch_bounds__(256, 6)
-causal_conv_norm_vec_kernel(const T* __restrict__ in, T* __restrict__ out, long long ld, long long out_ld, int col0,
+causal_conv_norm_vec_kernel(const T* __restrict__ in, TO* __restrict__ out, long long ld, long long out_ld, int col0,
                             int C, const float* __restrict__ taps, const float* __restrict__ state,
                             long long slot_stride, const int* __restrict__ tok_seg, const int* __restrict__ seg_start,
-                            const int* __restrict__ seg_slot, ConvNormRange r0, ConvNormRange r1, float eps) {
+                            const int* __restrict__ seg_slot, ConvNormRange r0, ConvNormRange r1, float eps,
+                            ConvFinish finish) {
     fwb::pdl_entry();
     extern __shared__ float4 row4[];               // [C / 4]
     __shared__ float scratch[66];
@@ -120,6 +131,7 @@ causal_conv_norm_vec_kernel(const T* __restrict__ in, T* __restrict__ out, long 
             acc.x = fmaf(w[j], u.x, acc.x), acc.y = fmaf(w[NT + j], u.y, acc.y);
             acc.z = fmaf(w[2 * NT + j], u.z, acc.z), acc.w = fmaf(w[3 * NT + j], u.w, acc.w);
         }
+        acc.x = finish(acc.x, c), acc.y = finish(acc.y, c + 1), acc.z = finish(acc.z, c + 2), acc.w = finish(acc.w, c + 3);
         row4[c >> 2] = acc;
         const float sq = fmaf(acc.x, acc.x, fmaf(acc.y, acc.y, fmaf(acc.z, acc.z, acc.w * acc.w)));
         if (c >= r0.col0 && c < r0.col0 + r0.width) ss0 += sq;
@@ -131,7 +143,7 @@ causal_conv_norm_vec_kernel(const T* __restrict__ in, T* __restrict__ out, long 
         inv0 = rsqrtf(sums.x / (float)(r0.count > 0 ? r0.count : 1) + eps);
         inv1 = rsqrtf(sums.y / (float)(r1.count > 0 ? r1.count : 1) + eps);
     }
-    T* dst = out + (size_t)t * out_ld;
+    TO* dst = out + (size_t)t * out_ld;
     for (int c = 4 * threadIdx.x; c < C; c += 4 * blockDim.x) {
         float4 v = row4[c >> 2];                   // (written by this very thread)
         if (c >= r0.col0 && c < r0.col0 + r0.width) {
@@ -141,18 +153,19 @@ causal_conv_norm_vec_kernel(const T* __restrict__ in, T* __restrict__ out, long 
             const float4 g = *reinterpret_cast<const float4*>(r1.weight + (c - r1.col0));
             v.x = (v.x * inv1) * g.x, v.y = (v.y * inv1) * g.y, v.z = (v.z * inv1) * g.z, v.w = (v.w * inv1) * g.w;
         }
-        store4<T>(dst + c, v);
+        store4<TO>(dst + c, v);
     }
 }
 
 // One block per token: the convolved row stays in shared memory while the sums of squares of its one or two
 // norm ranges are reduced, then every entry leaves scaled (entries outside the ranges leave as they are).
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
-causal_conv_norm_kernel(const T* __restrict__ in, T* __restrict__ out, long long ld, long long out_ld, int col0, int C,
+causal_conv_norm_kernel(const T* __restrict__ in, TO* __restrict__ out, long long ld, long long out_ld, int col0, int C,
                         const float* __restrict__ taps, int n, const float* __restrict__ state, long long slot_stride,
                         const int* __restrict__ tok_seg, const int* __restrict__ seg_start,
-                        const int* __restrict__ seg_slot, ConvNormRange r0, ConvNormRange r1, float eps) {
+                        const int* __restrict__ seg_slot, ConvNormRange r0, ConvNormRange r1, float eps,
+                            ConvFinish finish) {
     fwb::pdl_entry();
     extern __shared__ float row[];                 // [C]
     __shared__ float scratch[33];
@@ -162,7 +175,7 @@ causal_conv_norm_kernel(const T* __restrict__ in, T* __restrict__ out, long long
     const float* slot = state + (size_t)seg_slot[seg] * slot_stride;
     float ss0 = 0.0f, ss1 = 0.0f;
     for (int c = threadIdx.x; c < C; c += blockDim.x) {
-        const float v = conv_one<T>(in, (size_t)t * ld + col0 + c, ld, taps, n, c, C, local, slot);
+        const float v = finish(conv_one<T>(in, (size_t)t * ld + col0 + c, ld, taps, n, c, C, local, slot), c);
         row[c] = v;
         if (c >= r0.col0 && c < r0.col0 + r0.width) ss0 = fmaf(v, v, ss0);
         else if (c >= r1.col0 && c < r1.col0 + r1.width) ss1 = fmaf(v, v, ss1);
@@ -173,16 +186,16 @@ causal_conv_norm_kernel(const T* __restrict__ in, T* __restrict__ out, long long
         float v = row[c];
         if (c >= r0.col0 && c < r0.col0 + r0.width) v = (v * inv0) * r0.weight[c - r0.col0];
         else if (c >= r1.col0 && c < r1.col0 + r1.width) v = (v * inv1) * r1.weight[c - r1.col0];
-        out[(size_t)t * out_ld + c] = from_f32<T>(v);
+        out[(size_t)t * out_ld + c] = from_f32<TO>(v);
     }
 }
 
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(256)
-causal_conv_kernel(const T* __restrict__ in, T* __restrict__ out, long long ld, long long out_ld, int col0, int C,
+causal_conv_kernel(const T* __restrict__ in, TO* __restrict__ out, long long ld, long long out_ld, int col0, int C,
                    const float* __restrict__ taps, int n, const float* __restrict__ state, long long slot_stride,
                    const int* __restrict__ tok_seg, const int* __restrict__ seg_start,
-                   const int* __restrict__ seg_slot) {
+                   const int* __restrict__ seg_slot, ConvFinish finish) {
     fwb::pdl_entry();
     const int t = blockIdx.x;
     const int c = blockIdx.y * blockDim.x + threadIdx.x;
@@ -191,7 +204,7 @@ causal_conv_kernel(const T* __restrict__ in, T* __restrict__ out, long long ld, 
     const int local = t - seg_start[seg];                 // tokens of this segment in front of t
     const float* slot = state + (size_t)seg_slot[seg] * slot_stride;
     const float acc = conv_one<T>(in, (size_t)t * ld + col0 + c, ld, taps, n, c, C, local, slot);
-    out[(size_t)t * out_ld + c] = from_f32<T>(acc);
+    out[(size_t)t * out_ld + c] = from_f32<TO>(finish(acc, c));
 }
 
 // One thread per (segment, channel): the new state rows are the segment's last n - 1 inputs, or, for a
@@ -216,10 +229,10 @@ causal_conv_advance_kernel(const T* __restrict__ in, long long ld, int col0, int
     for (int k = 0; k < keep; ++k) slot[(size_t)k * C + c] = rows[k];
 }
 
-template <typename T>
+template <typename T, typename TO>
 int launch(const void* in, void* out, long long ld, long long out_ld, int col0, int C, const float* taps, int n,
            float* state, long long slot_stride, const int* tok_seg, const int* seg_start, const int* seg_slot,
-           int T_tokens, int S, ConvNormRange r0, ConvNormRange r1, float eps, cudaStream_t stream) {
+           int T_tokens, int S, ConvNormRange r0, ConvNormRange r1, float eps, ConvFinish finish, cudaStream_t stream) {
     const bool by_four = n <= 4 && C % 4 == 0 && ld % 4 == 0 && out_ld % 4 == 0 && col0 % 4 == 0 && r0.col0 % 4 == 0 &&
                          r0.width % 4 == 0 && r1.col0 % 4 == 0 && r1.width % 4 == 0 && (size_t)C * sizeof(float) <= 160 * 1024 &&
                          (((uintptr_t)in | (uintptr_t)out | (uintptr_t)taps | (uintptr_t)state | (uintptr_t)r0.weight |
@@ -229,11 +242,11 @@ int launch(const void* in, void* out, long long ld, long long out_ld, int col0, 
 #define FWB_CONV_VEC(NT)                                                                                          \
     do {                                                                                                          \
         if (smem > 48 * 1024)                                                                                     \
-            cudaFuncSetAttribute(causal_conv_norm_vec_kernel<T, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
+            cudaFuncSetAttribute(causal_conv_norm_vec_kernel<T, TO, NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, \
                                  (int)smem);                                                                      \
-        fwb::pdl(causal_conv_norm_vec_kernel<T, NT>, T_tokens, 256, smem, stream)(                                \
-            (const T*)in, (T*)out, ld, out_ld, col0, C, taps, state, slot_stride, tok_seg, seg_start, seg_slot,  \
-            r0, r1, eps);                                                                                         \
+        fwb::pdl(causal_conv_norm_vec_kernel<T, TO, NT>, T_tokens, 256, smem, stream)(                                \
+            (const T*)in, (TO*)out, ld, out_ld, col0, C, taps, state, slot_stride, tok_seg, seg_start, seg_slot, \
+            r0, r1, eps, finish);                                                                                         \
     } while (0)
         switch (n) {
             case 1: FWB_CONV_VEC(1); break;
@@ -245,14 +258,14 @@ int launch(const void* in, void* out, long long ld, long long out_ld, int col0, 
     } else if (r0.width > 0) {
         const size_t smem = (size_t)C * sizeof(float);
         if (smem > 48 * 1024)
-            cudaFuncSetAttribute(causal_conv_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-        fwb::pdl(causal_conv_norm_kernel<T>, T_tokens, 256, smem, stream)(
-            (const T*)in, (T*)out, ld, out_ld, col0, C, taps, n, state, slot_stride, tok_seg, seg_start, seg_slot, r0,
-            r1, eps);
+            cudaFuncSetAttribute(causal_conv_norm_kernel<T, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        fwb::pdl(causal_conv_norm_kernel<T, TO>, T_tokens, 256, smem, stream)(
+            (const T*)in, (TO*)out, ld, out_ld, col0, C, taps, n, state, slot_stride, tok_seg, seg_start, seg_slot, r0,
+            r1, eps, finish);
     } else {
         const dim3 grid(T_tokens, (C + 255) / 256);
-        fwb::pdl(causal_conv_kernel<T>, grid, 256, 0, stream)((const T*)in, (T*)out, ld, out_ld, col0, C, taps, n,
-                                                              state, slot_stride, tok_seg, seg_start, seg_slot);
+        fwb::pdl(causal_conv_kernel<T, TO>, grid, 256, 0, stream)((const T*)in, (TO*)out, ld, out_ld, col0, C, taps, n,
+                                                                  state, slot_stride, tok_seg, seg_start, seg_slot, finish);
     }
     if (n > 1) {
         const dim3 grid2(S, (C + 255) / 256);
@@ -264,11 +277,12 @@ int launch(const void* in, void* out, long long ld, long long out_ld, int col0, 
 
 }  // namespace
 
-// in: [T][ld], out: [T][out_ld], fp32 or bf16 (both of one type, different buffers); taps: [C][n] fp32; state: fp32,
+// in: [T][ld], out: [T][out_ld], fp32 or bf16 (different buffers; bf16 to fp32 has no form); bias: fp32 [C] or null;
+// silu: 0 or 1; taps: [C][n] fp32; state: fp32,
 // slot s at state + s * slot_stride, [n - 1][C] (may be null when n == 1); tok_seg: [T]; seg_start: [S + 1];
 // seg_slot: [S].  Norm ranges (width0 == 0: none; width1 == 0: one): columns [c0, c0 + width) of the output, the
 // mean of squares over `count` channels, weights fp32 [width].
-FWB_API int fwb_causal_conv(const void* in, void* out, int is_bf16, long long ld, long long out_ld, int col0, int C,
+FWB_API int fwb_causal_conv(const void* in, void* out, int is_bf16, int out_bf16, const float* bias, int silu, long long ld, long long out_ld, int col0, int C,
                             const float* taps, int n, float* state, long long slot_stride, const int* tok_seg,
                             const int* seg_start, const int* seg_slot, int T, int S, int norm_col0, int norm_width0,
                             int norm_count0, const float* norm_w0, int norm_col1, int norm_width1, int norm_count1,
@@ -287,8 +301,13 @@ FWB_API int fwb_causal_conv(const void* in, void* out, int is_bf16, long long ld
     } else if (r1.width > 0) {
         return FWB_BAD_ARGUMENT;
     }
-    return is_bf16 ? launch<__nv_bfloat16>(in, out, ld, out_ld, col0, C, taps, n, state, slot_stride, tok_seg, seg_start,
-                                           seg_slot, T, S, r0, r1, eps, stream)
-                   : launch<float>(in, out, ld, out_ld, col0, C, taps, n, state, slot_stride, tok_seg, seg_start,
-                                   seg_slot, T, S, r0, r1, eps, stream);
+    if (is_bf16 && !out_bf16) return FWB_UNSUPPORTED;
+    const ConvFinish finish{bias, silu};
+    if (!is_bf16 && out_bf16)
+        return launch<float, __nv_bfloat16>(in, out, ld, out_ld, col0, C, taps, n, state, slot_stride, tok_seg, seg_start,
+                                            seg_slot, T, S, r0, r1, eps, finish, stream);
+    return is_bf16 ? launch<__nv_bfloat16, __nv_bfloat16>(in, out, ld, out_ld, col0, C, taps, n, state, slot_stride, tok_seg, seg_start,
+                                           seg_slot, T, S, r0, r1, eps, finish, stream)
+                   : launch<float, float>(in, out, ld, out_ld, col0, C, taps, n, state, slot_stride, tok_seg, seg_start,
+                                   seg_slot, T, S, r0, r1, eps, finish, stream);
 }

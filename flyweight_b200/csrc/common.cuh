@@ -170,8 +170,8 @@ __device__ __forceinline__ float silu_f32(float g) {
 
 // What a gated feed-forward makes of a gate value g and an up value u.  0: silu(g) u.  1: gelu(g) u (tanh
 // form).  2, the clamped swish: g is cut off above `limit`, u is held inside [-limit, limit], and the
-// result is g sigmoid(1.702 g) (u + 1).
-constexpr int GATED_SILU = 0, GATED_GELU_TANH = 1, GATED_SWISH_CLAMPED = 2;
+// result is g sigmoid(1.702 g) (u + 1).  3: max(g, 0) u.
+constexpr int GATED_SILU = 0, GATED_GELU_TANH = 1, GATED_SWISH_CLAMPED = 2, GATED_RELU = 3;
 constexpr float SWISH_CLAMPED_SLOPE = 1.702f;
 __device__ __forceinline__ float gated_f32(int act, float limit, float g, float u) {
     if (act == GATED_SWISH_CLAMPED) {
@@ -182,7 +182,16 @@ __device__ __forceinline__ float gated_f32(int act, float limit, float g, float 
         const float sig = z >= 0.0f ? 1.0f / (1.0f + e) : e / (1.0f + e);
         return g * sig * (u + 1.0f);
     }
+    if (act == GATED_RELU) return fmaxf(g, 0.0f) * u;
     return (act == GATED_GELU_TANH ? gelu_tanh_f32(g) : silu_f32(g)) * u;
+}
+
+// What a product without a gate may do to its output before it is stored.  0: nothing.  1: max(v, 0)^2.
+constexpr int OUTPUT_AS_IS = 0, OUTPUT_RELU_SQUARED = 1;
+__device__ __forceinline__ float output_act_f32(int act, float v) {
+    if (act != OUTPUT_RELU_SQUARED) return v;
+    const float r = fmaxf(v, 0.0f);
+    return r * r;
 }
 
 }  // namespace fwb

@@ -104,7 +104,7 @@ struct Params {
     int M, N, K;           // tokens, features (of one accumulator), reduction
     int ldy;
     int up_row_offset;     // SwiGLU: rows of the up projection start here in W
-    int gate_act;          // SwiGLU: the gate's activation (tc5 GATE_SILU | GATE_GELU_TANH | GATE_SWISH_CLAMPED)
+    int gate_act;          // SwiGLU: the gate's activation (tc5 GATE_*); bf16 outputs: what is done to them (OUTPUT_*)
     float gate_limit;      // the clamped swish's limit
     int k_blocks_per_split;
     int stages;            // depth of the shared-memory ring (<= Tile::MAX_STAGES)
@@ -373,10 +373,11 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_cons
             reinterpret_cast<float*>(prm.y)[at] = g;
             if (f + BM < prm.N) reinterpret_cast<float*>(prm.y)[at + BM] = u;
         } else if (EPI == EPI_BF16_WIDE) {
-            reinterpret_cast<__nv_bfloat16*>(prm.y)[at] = __float2bfloat16_rn(g);
-            if (f + BM < prm.N) reinterpret_cast<__nv_bfloat16*>(prm.y)[at + BM] = __float2bfloat16_rn(u);
+            reinterpret_cast<__nv_bfloat16*>(prm.y)[at] = __float2bfloat16_rn(output_act_f32(prm.gate_act, g));
+            if (f + BM < prm.N)
+                reinterpret_cast<__nv_bfloat16*>(prm.y)[at + BM] = __float2bfloat16_rn(output_act_f32(prm.gate_act, u));
         } else if (EPI == EPI_ADD_F32) reinterpret_cast<float*>(prm.y)[at] = g + (splits > 1 ? u : prm.addend[at]);
-        else if (EPI == EPI_BF16) reinterpret_cast<__nv_bfloat16*>(prm.y)[at] = __float2bfloat16_rn(g);
+        else if (EPI == EPI_BF16) reinterpret_cast<__nv_bfloat16*>(prm.y)[at] = __float2bfloat16_rn(output_act_f32(prm.gate_act, g));
         else reinterpret_cast<__nv_bfloat16*>(prm.y)[at] = __float2bfloat16_rn(gated_fast(prm.gate_act, prm.gate_limit, g, u));
     };
 
@@ -549,7 +550,7 @@ int launch_epi(int epi, const CUtensorMap& map_w, const CUtensorMap& map_x, cons
 FWB_API int fwb_gemm_tcgen05(const void* X, const void* W, void* Y, const float* addend, int M, int N,
                              int K, int w_rows, int ldy, int epilogue, int up_row_offset, int splits,
                              int stages, int tile_tokens, int wide, float gate_limit, cudaStream_t stream) {
-    const int gate_act = epilogue >> 8;     // bits above the epilogue code: the gate's activation
+    const int gate_act = epilogue >> 8;     // bits above the epilogue code: the gate's, or a bf16 output's, activation
     epilogue &= 0xff;
     if (M <= 0 || N <= 0) return FWB_OK;
     if (!X || !W || !Y || K <= 0 || ldy < N) return FWB_BAD_ARGUMENT;

@@ -53,7 +53,7 @@ struct PairParams {
     void* y;
     int M, N, K, ldy;
     int up_row_offset;
-    int gate_act;          // SwiGLU: the gate's activation (GATE_SILU | GATE_GELU_TANH)
+    int gate_act;          // SwiGLU: the gate's activation (GATE_SILU | GATE_GELU_TANH); bf16 outputs: OUTPUT_*
     int token_tiles;
     int* status;
 };
@@ -229,16 +229,18 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constan
                     if (t >= prm.M || f >= prm.N) continue;
                     const size_t at = (size_t)t * prm.ldy + f;
                     if (EPI == PAIR_F32) reinterpret_cast<float*>(prm.y)[at] = g[j];
-                    else if (EPI == PAIR_BF16) reinterpret_cast<__nv_bfloat16*>(prm.y)[at] = __float2bfloat16_rn(g[j]);
+                    else if (EPI == PAIR_BF16)
+                        reinterpret_cast<__nv_bfloat16*>(prm.y)[at] = __float2bfloat16_rn(output_act_f32(prm.gate_act, g[j]));
                     else if (EPI == PAIR_SWIGLU_BF16)
                         reinterpret_cast<__nv_bfloat16*>(prm.y)[at] = __float2bfloat16_rn(gate_act_fast(prm.gate_act, g[j]) * u[j]);
                     else if (EPI == PAIR_F32_WIDE) {
                         reinterpret_cast<float*>(prm.y)[at] = g[j];
                         if (f + PAIR_M < prm.N) reinterpret_cast<float*>(prm.y)[at + PAIR_M] = u[j];
                     } else {
-                        reinterpret_cast<__nv_bfloat16*>(prm.y)[at] = __float2bfloat16_rn(g[j]);
+                        reinterpret_cast<__nv_bfloat16*>(prm.y)[at] = __float2bfloat16_rn(output_act_f32(prm.gate_act, g[j]));
                         if (f + PAIR_M < prm.N)
-                            reinterpret_cast<__nv_bfloat16*>(prm.y)[at + PAIR_M] = __float2bfloat16_rn(u[j]);
+                            reinterpret_cast<__nv_bfloat16*>(prm.y)[at + PAIR_M] =
+                                __float2bfloat16_rn(output_act_f32(prm.gate_act, u[j]));
                     }
                 }
             }
@@ -286,7 +288,7 @@ int launch(const CUtensorMap& map_w, const CUtensorMap& map_x, const PairParams&
 // CTA pair two blocks of 256 features (plain epilogues only).  K % 8 == 0, bases 16-byte aligned.
 FWB_API int fwb_gemm_tcgen05_pair(const void* X, const void* W, void* Y, int M, int N, int K, int w_rows,
                                   int ldy, int epilogue, int up_row_offset, int wide, cudaStream_t stream) {
-    const int gate_act = epilogue >> 8;     // bits above the epilogue code: the gate's activation
+    const int gate_act = epilogue >> 8;     // bits above the epilogue code: the gate's, or a bf16 output's, activation
     epilogue &= 0xff;
     if (gate_act > GATE_GELU_TANH) return FWB_UNSUPPORTED;     // (activations with a parameter: the one-CTA kernel)
     if (M <= 0 || N <= 0) return FWB_OK;

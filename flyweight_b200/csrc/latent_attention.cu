@@ -16,6 +16,8 @@
 // Kernels of this file:
 //   fwb_latent_prepare    rotation of the queries' rotated part, RMS norm of the latent, rotation of
 //                         the shared key part, write of the cache row (one pass over the projection)
+//   fwb_latent_low_rank   for a model whose queries come from a low-rank row as well: both RMS norms (the
+//                         queries' row, the latent), rotation of the shared key part, write of the cache row
 //   fwb_head_linear       Y[t][h] = W[h] X[t][h] for every head, fp32 FMA (any sizes, any strides)
 //   fwb_latent_attention_simt   the attention in fp32 arithmetic, any sizes: the 32-bit path
 // In bfloat16 the per-head products run on tensor cores (head_linear_mma.cu) and the attention on the
@@ -86,6 +88,60 @@ __global__ void latent_prepare_kernel(const TP* __restrict__ proj, int ld, int k
         float v = 0.0f;
         if (c < rank) v = (to_f32<TP>(lat[c]) * inv) * norm_w[c];
         else if (c < rank + rot) v = turned(lat + rank, c - rank);
+        dst[c] = from_f32<TC>(v);
+    }
+}
+
+// One block per token.  proj: [T][ld] rows [ queries' row (q_rank) | latent (rank) | shared key part (rot) ]; both
+// rows are brought to unit root mean square and weighted; the queries' goes to cq [T][q_rank] (the next
+// product's input), the latent with the turned key part and zero padding into the token's cache row.
+template <typename TP, typename TQ, typename TC>
+__global__ void latent_low_rank_kernel(const TP* __restrict__ proj, int ld, int q_rank,
+                                       const float* __restrict__ q_norm_w, const float* __restrict__ norm_w,
+                                       const float* __restrict__ table, const int* __restrict__ positions,
+                                       const int* __restrict__ tok_seg, const int* __restrict__ block_table,
+                                       int max_pages, int page_size, TQ* __restrict__ cq, TC* __restrict__ pool,
+                                       int rot, int rot_dims, int interleaved, int rank, int row, float eps) {
+    fwb::pdl_entry();
+    __shared__ float scratch[33];
+    const int t = blockIdx.x;
+    const TP* src = proj + (size_t)t * ld;
+    float ss = 0.0f;
+    for (int c = threadIdx.x; c < q_rank; c += blockDim.x) {
+        const float v = to_f32<TP>(src[c]);
+        ss = fmaf(v, v, ss);
+    }
+    const float inv_q = rsqrtf(block_sum(ss, scratch) / (float)q_rank + eps);
+    for (int c = threadIdx.x; c < q_rank; c += blockDim.x)
+        cq[(size_t)t * q_rank + c] = from_f32<TQ>((to_f32<TP>(src[c]) * inv_q) * q_norm_w[c]);
+    if (!pool) return;
+    const int pos = positions[t];
+    const int half = rot_dims >> 1;
+    const float* cs = table + (size_t)pos * (half > 0 ? half : 1) * 2;
+    const TP* lat = src + q_rank;
+    ss = 0.0f;
+    for (int c = threadIdx.x; c < rank; c += blockDim.x) {
+        const float v = to_f32<TP>(lat[c]);
+        ss = fmaf(v, v, ss);
+    }
+    const float inv = rsqrtf(block_sum(ss, scratch) / (float)rank + eps);
+    const int page = block_table[(size_t)tok_seg[t] * max_pages + pos / page_size];
+    TC* dst = pool + ((size_t)page * page_size + (pos % page_size)) * row;
+    for (int c = threadIdx.x; c < row; c += blockDim.x) {
+        float v = 0.0f;
+        if (c < rank) {
+            v = (to_f32<TP>(lat[c]) * inv) * norm_w[c];
+        } else if (c < rank + rot) {
+            const TP* part = lat + rank;
+            const int i = c - rank;
+            v = to_f32<TP>(part[i]);
+            if (i < rot_dims) {
+                const int pair = interleaved ? i >> 1 : (i < half ? i : i - half);
+                const int partner = interleaved ? i ^ 1 : (i < half ? i + half : i - half);
+                const float sign = (interleaved ? (i & 1) == 0 : i < half) ? -1.0f : 1.0f;
+                v = v * cs[2 * pair] + sign * to_f32<TP>(part[partner]) * cs[2 * pair + 1];
+            }
+        }
         dst[c] = from_f32<TC>(v);
     }
 }
@@ -266,6 +322,32 @@ FWB_API int fwb_latent_prepare(const void* proj, int proj_bf16, int ld, int kv_c
     else if (proj_bf16) FWB_PREP(bf, float);
     else FWB_PREP(float, bf);
 #undef FWB_PREP
+    return fwb_launch_status();
+}
+
+// proj: [T][ld] (fp32 or bf16), ld >= q_rank + rank + rot; cq: [T][q_rank]; pool: [pages][page_size][row] or null
+// (the queries' row only).
+FWB_API int fwb_latent_low_rank(const void* proj, int proj_bf16, int ld, int q_rank, const float* q_norm_w,
+                                const float* norm_w, const float* table, const int* positions, const int* tok_seg,
+                                const int* block_table, int max_pages, int page_size, void* cq, int cq_bf16, void* pool,
+                                int pool_bf16, int T, int rot, int rot_dims, int interleaved, int rank, int row,
+                                float eps, cudaStream_t stream) {
+    if (T <= 0) return FWB_OK;
+    if (!proj || !q_norm_w || !cq || q_rank <= 0 || ld < q_rank) return FWB_BAD_ARGUMENT;
+    if (rot < 0 || rank <= 0 || row < rank + rot || rot_dims < 0 || rot_dims > rot || (rot_dims & 1)) return FWB_BAD_ARGUMENT;
+    if (pool && (!norm_w || !table || !positions || !tok_seg || !block_table || max_pages <= 0 || page_size <= 0
+                 || ld < q_rank + rank + rot))
+        return FWB_BAD_ARGUMENT;
+    using bf = __nv_bfloat16;
+#define FWB_LOW_RANK(TP, TQ, TC)                                                                              \
+    fwb::pdl(latent_low_rank_kernel<TP, TQ, TC>, T, 256, 0, stream)(                                          \
+        (const TP*)proj, ld, q_rank, q_norm_w, norm_w, table, positions, tok_seg, block_table, max_pages,    \
+        page_size, (TQ*)cq, (TC*)pool, rot, rot_dims, interleaved, rank, row, eps)
+    if (proj_bf16 && cq_bf16 && (pool_bf16 || !pool)) FWB_LOW_RANK(bf, bf, bf);
+    else if (!proj_bf16 && cq_bf16 && (pool_bf16 || !pool)) FWB_LOW_RANK(float, bf, bf);
+    else if (!proj_bf16 && !cq_bf16 && !pool_bf16) FWB_LOW_RANK(float, float, float);
+    else return FWB_UNSUPPORTED;
+#undef FWB_LOW_RANK
     return fwb_launch_status();
 }
 

@@ -6,13 +6,17 @@
 //            is its largest choice value, only the `keep` best runs stay in the race (the others count
 //            as minus infinity), and the `top` largest survivors are chosen.  The weights are the plain
 //            s of the chosen, not renormalised.  Ties go to the lower index.
-//            Optionally s = sigmoid(router h) instead, each output on its own, and no correction.
+//            Optionally s = sigmoid(router h) instead, each output on its own, and no correction; or the choice
+//            is made on the outputs themselves, router h + correction, and the weights are the softmax over the
+//            chosen outputs alone.  The router's matrix may carry one row more than it has outputs: its
+//            sigmoid is handed out per token (the gate of an expert that every token shares).
 //   sort     pairs whose output is a real expert (index < E) are counted per expert, the counts are
 //            scanned, every pair gets its row among its expert's rows, and the row tiles of the two
 //            products are listed.  Outputs from E on are identity experts: they have no row.
 //   gemm     one CTA per (row tile of one expert, tile of output features): rows gathered through the
 //            sorted list, fp32 FMA accumulation over k in order.  Form 1: act(x gate^T) * (x up^T) for
-//            the stacked matrix [gate rows | up rows]; form 0: the plain product in fp32.
+//            the stacked matrix [gate rows | up rows]; form 2: act(x w^T) without a gate; form 0: the plain
+//            product in fp32.
 //   gather   the sorted rows' inputs side by side, for the grouped tensor-core product (bfloat16)
 //   combine  out[t] = sum over the token's pairs, in slot order, of weight * (expert row | h[t] itself
 //            for an identity expert); with weights that belong on the experts' inputs the rows were
@@ -29,7 +33,8 @@ using namespace fwb;
 namespace {
 
 constexpr int TM = 64, TN = 64, TK = 16;       // tile of the experts' products
-constexpr int SCORE_SIGMOID = 1;               // a router's scores: 0 softmax over the outputs, 1 sigmoid of each
+// a router's scores: 0 softmax over the outputs, 1 sigmoid of each, 2 softmax over the chosen outputs alone
+constexpr int SCORE_SIGMOID = 1, SCORE_SOFTMAX_CHOSEN = 2;
 
 // One warp: from a token's router outputs s[N] (shared memory) to its scores, the choice inside the kept runs,
 // and the `top` chosen outputs with their scores.  choice[N], best[n_groups]: scratch in shared memory.
@@ -42,6 +47,9 @@ __device__ __forceinline__ void choose_outputs(float* s, float* choice, float* b
             const float z = s[n], e = expf(-fabsf(z));
             s[n] = z >= 0.0f ? 1.0f / (1.0f + e) : e / (1.0f + e);
         }
+    } else if (scoring == SCORE_SOFTMAX_CHOSEN) {
+        for (int n = lane; n < N; n += 32) s[n] += correction ? correction[n] : 0.0f;
+        correction = nullptr;                      // (part of the outputs from here on)
     } else {
         float m = -INFINITY;
         for (int n = lane; n < N; n += 32) m = fmaxf(m, s[n]);
@@ -110,16 +118,29 @@ __device__ __forceinline__ void choose_outputs(float* s, float* choice, float* b
         }
         __syncwarp();
     }
+    if (scoring == SCORE_SOFTMAX_CHOSEN && lane == 0) {
+        const float m = weights[0];                // the largest: it was chosen first
+        float sum = 0.0f;
+        for (int slot = 0; slot < top; ++slot) sum += expf(weights[slot] - m);
+        for (int slot = 0; slot < top; ++slot) weights[slot] = expf(weights[slot] - m) / sum;
+    }
+}
+
+__device__ __forceinline__ float sigmoid_of(float z) {
+    const float e = expf(-fabsf(z));
+    return z >= 0.0f ? 1.0f / (1.0f + e) : e / (1.0f + e);
 }
 
 template <typename TH>
 __global__ void __launch_bounds__(512)
 moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, const float* __restrict__ correction,
-                 int* __restrict__ ids, float* __restrict__ weights, int T, int W, int N, int n_groups, int keep,
-                 int top, int vec, int scoring) {
+                 int* __restrict__ ids, float* __restrict__ weights, int T, int W, int N_choice, int n_groups, int keep,
+                 int top, int vec, int scoring, float* __restrict__ gate_out) {
     fwb::pdl_entry();
     // One block per token.  Its warps share the router's outputs between them (output n: lanes stride
     // over k with sixteen sums in flight, added in one fixed order); warp 0 then chooses.
+    // `gate_out`: the matrix has a row behind the outputs', whose sigmoid goes there.
+    const int N = N_choice + (gate_out ? 1 : 0);  // rows of the matrix
     extern __shared__ float shared[];             // s[N], choice[N], group value[n_groups]
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x;
@@ -206,20 +227,24 @@ moe_route_kernel(const TH* __restrict__ h, const float* __restrict__ router, con
     }
     __syncthreads();
     if (warp != 0) return;
-    choose_outputs(s, choice, best, correction, ids + (size_t)t * top, weights + (size_t)t * top, N, n_groups, keep, top, scoring);
+    if (gate_out && lane == 0) gate_out[t] = sigmoid_of(s[N_choice]);
+    choose_outputs(s, choice, best, correction, ids + (size_t)t * top, weights + (size_t)t * top, N_choice, n_groups, keep, top,
+                   scoring);
 }
 
 // The choice alone, from router outputs that a matrix product made: one warp a token.
 __global__ void __launch_bounds__(128)
 moe_choose_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int* __restrict__ ids,
-                  float* __restrict__ weights, int T, int N, int n_groups, int keep, int top, int scoring) {
+                  float* __restrict__ weights, int T, int N, int n_groups, int keep, int top, int scoring,
+                  long long ld, float* __restrict__ gate_out) {
     fwb::pdl_entry();
     extern __shared__ float shared[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int t = blockIdx.x * (blockDim.x >> 5) + warp;
     if (t >= T) return;
     float* s = shared + warp * (2 * N + n_groups);
-    for (int n = lane; n < N; n += 32) s[n] = logits[(size_t)t * N + n];
+    for (int n = lane; n < N; n += 32) s[n] = logits[(size_t)t * ld + n];
+    if (gate_out && lane == 0) gate_out[t] = sigmoid_of(logits[(size_t)t * ld + N]);
     __syncwarp();
     choose_outputs(s, s + N, s + 2 * N, correction, ids + (size_t)t * top, weights + (size_t)t * top, N, n_groups, keep, top,
                    scoring);
@@ -349,8 +374,9 @@ moe_gather_rows_kernel(const uint4* __restrict__ h, const int* __restrict__ row_
 }
 
 // FORM 1: out[row][f] = act(x . gate_f) * (x . up_f), w: [E][2F][K] (gate rows, then up rows), N = F.
+// FORM 2: out[row][f] = act(x . w_f), w: [E][F][K], N = F (act: an OUTPUT_* code).
 // FORM 0: out[row][n] = x . w_n, w: [E][N][K], fp32 out.
-// x rows: FORM 1 gathers token rows through row_token; FORM 0 reads sorted rows directly.
+// x rows: FORMs 1 and 2 gather token rows through row_token; FORM 0 reads sorted rows directly.
 template <typename TX, typename TW, typename TO, int FORM>
 __global__ void __launch_bounds__(256)
 moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TO* __restrict__ out,
@@ -363,7 +389,7 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TO* __restri
     const int row_end = offsets[expert + 1];
     const int n0 = blockIdx.x * TN;
     __shared__ float xs[TK][TM + 1];
-    __shared__ float ws[FORM ? 2 : 1][TK][TN + 1];
+    __shared__ float ws[FORM == 1 ? 2 : 1][TK][TN + 1];
     __shared__ int src_row[TM];
     __shared__ float src_weight[TM];              // what the row's input is multiplied by (FORM 1)
     if (threadIdx.x < TM) {
@@ -372,7 +398,7 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TO* __restri
         src_row[threadIdx.x] = row < row_end ? (FORM ? row_token[row] : row) : -1;
     }
     __syncthreads();
-    const TW* w_gate = w + (size_t)expert * (FORM ? 2 : 1) * N * K;
+    const TW* w_gate = w + (size_t)expert * (FORM == 1 ? 2 : 1) * N * K;
     const TW* w_up = w_gate + (size_t)N * K;
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;      // 16 x 16 threads, 4 x 4 outputs each
     float acc[4][4] = {}, acc2[4][4] = {};
@@ -387,7 +413,7 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TO* __restri
             const int n = i / TK, k = i - n * TK;
             const bool in = n0 + n < N && k0 + k < K;
             ws[0][k][n] = in ? to_f32<TW>(w_gate[(size_t)(n0 + n) * K + k0 + k]) : 0.0f;
-            if (FORM) ws[1][k][n] = in ? to_f32<TW>(w_up[(size_t)(n0 + n) * K + k0 + k]) : 0.0f;
+            if (FORM == 1) ws[1][k][n] = in ? to_f32<TW>(w_up[(size_t)(n0 + n) * K + k0 + k]) : 0.0f;
         }
         __syncthreads();
 #pragma unroll
@@ -398,14 +424,14 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TO* __restri
 #pragma unroll
             for (int j = 0; j < 4; ++j) {
                 b[j] = ws[0][k][tx * 4 + j];
-                if (FORM) b2[j] = ws[1][k][tx * 4 + j];
+                if (FORM == 1) b2[j] = ws[1][k][tx * 4 + j];
             }
 #pragma unroll
             for (int i = 0; i < 4; ++i)
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
-                    if (FORM) acc2[i][j] = fmaf(a[i], b2[j], acc2[i][j]);
+                    if (FORM == 1) acc2[i][j] = fmaf(a[i], b2[j], acc2[i][j]);
                 }
         }
         __syncthreads();
@@ -419,7 +445,8 @@ moe_gemm_kernel(const TX* __restrict__ x, const TW* __restrict__ w, TO* __restri
             const int n = n0 + tx * 4 + j;
             if (n >= N) continue;
             float v = acc[i][j];
-            if (FORM) v = gated_f32(act, limit, v, acc2[i][j]);
+            if (FORM == 1) v = gated_f32(act, limit, v, acc2[i][j]);
+            if (FORM == 2) v = output_act_f32(act, v);
             out[(size_t)row * N + n] = from_f32<TO>(v);
         }
     }
@@ -429,7 +456,7 @@ template <typename TH>
 __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ y, const TH* __restrict__ h, const int* __restrict__ pair_row,
                    const int* __restrict__ ids, const float* __restrict__ weights, float* __restrict__ out, int W,
-                   int top, int E, int weighted_in) {
+                   int top, int E, const float* __restrict__ extra, const float* __restrict__ extra_gate, int weighted_in) {
     fwb::pdl_entry();
     constexpr int MAX_TOP = 64;
     __shared__ int rows[MAX_TOP];                 // the sorted row of every slot; -1: identity; -2: nothing
@@ -442,6 +469,7 @@ moe_combine_kernel(const float* __restrict__ y, const TH* __restrict__ h, const 
         wts[threadIdx.x] = weighted_in && row >= 0 ? 1.0f : weights[a];
     }
     __syncthreads();
+    const float extra_scale = extra_gate ? extra_gate[t] : 1.0f;
     if ((W & 3) == 0 && sizeof(TH) == 4) {
         // rows of 16-byte pieces (the fp32 path's h as well as y)
         const float4* y4 = reinterpret_cast<const float4*>(y);
@@ -455,6 +483,11 @@ moe_combine_kernel(const float* __restrict__ y, const TH* __restrict__ h, const 
                 const float wt = wts[slot];
                 acc.x = fmaf(wt, v.x, acc.x), acc.y = fmaf(wt, v.y, acc.y);
                 acc.z = fmaf(wt, v.z, acc.z), acc.w = fmaf(wt, v.w, acc.w);
+            }
+            if (extra) {
+                const float4 more = reinterpret_cast<const float4*>(extra)[(size_t)t * (W / 4) + i];
+                acc.x = fmaf(extra_scale, more.x, acc.x), acc.y = fmaf(extra_scale, more.y, acc.y);
+                acc.z = fmaf(extra_scale, more.z, acc.z), acc.w = fmaf(extra_scale, more.w, acc.w);
             }
             reinterpret_cast<float4*>(out)[(size_t)t * (W / 4) + i] = acc;
         }
@@ -478,6 +511,11 @@ moe_combine_kernel(const float* __restrict__ y, const TH* __restrict__ h, const 
                 acc.x = fmaf(wt, v.x, acc.x), acc.y = fmaf(wt, v.y, acc.y);
                 acc.z = fmaf(wt, v.z, acc.z), acc.w = fmaf(wt, v.w, acc.w);
             }
+            if (extra) {
+                const float4 more = reinterpret_cast<const float4*>(extra)[(size_t)t * (W / 4) + i];
+                acc.x = fmaf(extra_scale, more.x, acc.x), acc.y = fmaf(extra_scale, more.y, acc.y);
+                acc.z = fmaf(extra_scale, more.z, acc.z), acc.w = fmaf(extra_scale, more.w, acc.w);
+            }
             reinterpret_cast<float4*>(out)[(size_t)t * (W / 4) + i] = acc;
         }
         return;
@@ -500,6 +538,7 @@ moe_combine_kernel(const float* __restrict__ y, const TH* __restrict__ h, const 
             }
             acc = fmaf(wts[slot], v, acc);
         }
+        if (extra) acc = fmaf(extra_scale, extra[(size_t)t * W + i], acc);
         out[(size_t)t * W + i] = acc;
     }
 }
@@ -512,7 +551,7 @@ __global__ void __launch_bounds__(256)
 moe_combine_norm_add_kernel(const float* __restrict__ y, const TH* __restrict__ h, const int* __restrict__ pair_row,
                             const int* __restrict__ ids, const float* __restrict__ weights, float* __restrict__ x,
                             const float* __restrict__ norm_w, float eps, int W, int top, int E,
-                            const float* __restrict__ extra, int weighted_in) {
+                            const float* __restrict__ extra, const float* __restrict__ extra_gate, int weighted_in) {
     fwb::pdl_entry();
     constexpr int MAX_TOP = 64;
     extern __shared__ float sum_row[];            // [W]
@@ -527,6 +566,7 @@ moe_combine_norm_add_kernel(const float* __restrict__ y, const TH* __restrict__ 
         wts[threadIdx.x] = weighted_in && row >= 0 ? 1.0f : weights[a];
     }
     __syncthreads();
+    const float extra_scale = extra_gate ? extra_gate[t] : 1.0f;
     float ss = 0.0f;
     if ((W & 3) == 0) {
         // rows of 16-byte pieces; every element is still its own sum over the slots, in slot order
@@ -544,7 +584,8 @@ moe_combine_norm_add_kernel(const float* __restrict__ y, const TH* __restrict__ 
             }
             if (extra) {                               // (what every token gets besides its experts: added last)
                 const float4 more = reinterpret_cast<const float4*>(extra)[(size_t)t * (W / 4) + i];
-                acc.x += more.x, acc.y += more.y, acc.z += more.z, acc.w += more.w;
+                acc.x = fmaf(extra_scale, more.x, acc.x), acc.y = fmaf(extra_scale, more.y, acc.y);
+                acc.z = fmaf(extra_scale, more.z, acc.z), acc.w = fmaf(extra_scale, more.w, acc.w);
             }
             reinterpret_cast<float4*>(sum_row)[i] = acc;
             ss = fmaf(acc.x, acc.x, fmaf(acc.y, acc.y, fmaf(acc.z, acc.z, fmaf(acc.w, acc.w, ss))));
@@ -558,7 +599,7 @@ moe_combine_norm_add_kernel(const float* __restrict__ y, const TH* __restrict__ 
                 const float v = row >= 0 ? y[(size_t)row * W + i] : (row == -1 ? own : 0.0f);
                 acc = fmaf(wts[slot], v, acc);
             }
-            if (extra) acc += extra[(size_t)t * W + i];
+            if (extra) acc = fmaf(extra_scale, extra[(size_t)t * W + i], acc);
             sum_row[i] = acc;
             ss = fmaf(acc, acc, ss);
         }
@@ -570,12 +611,13 @@ moe_combine_norm_add_kernel(const float* __restrict__ y, const TH* __restrict__ 
 }  // namespace
 
 // h: [T][W] fp32 or bf16; router: [N][W] fp32; correction: [N] fp32 or null; ids, weights: [T][top].
-// scoring: 0 softmax over the outputs, 1 the sigmoid of each.
+// scoring: 0 softmax over the outputs, 1 the sigmoid of each, 2 softmax over the chosen outputs alone.
+// gate_out: [T] or null; with it the router's matrix is [N + 1][W] and the last row's sigmoid goes there.
 FWB_API int fwb_moe_route(const void* h, int h_bf16, const float* router, const float* correction, int* ids,
                           float* weights, int T, int W, int N, int n_groups, int keep, int top, int scoring,
-                          cudaStream_t stream) {
+                          float* gate_out, cudaStream_t stream) {
     if (T <= 0) return FWB_OK;
-    if (!h || !router || !ids || !weights || scoring < 0 || scoring > 1) return FWB_BAD_ARGUMENT;
+    if (!h || !router || !ids || !weights || scoring < 0 || scoring > 2) return FWB_BAD_ARGUMENT;
     if (W <= 0 || N <= 0 || n_groups <= 0 || N % n_groups || keep <= 0 || keep > n_groups || top <= 0 ||
         top > keep * (N / n_groups))
         return FWB_BAD_ARGUMENT;
@@ -586,28 +628,31 @@ FWB_API int fwb_moe_route(const void* h, int h_bf16, const float* router, const 
     // 115 us against 155 the other way).
     const int vec = (W % 4 == 0 && ((uintptr_t)router & 15) == 0 && W >= 512 && T < 256) ? 1 : 0;
     const int threads = vec ? 512 : (N >= 32 ? 512 : (N >= 16 ? 256 : 128));
-    const size_t smem = (size_t)(2 * N + n_groups + (vec ? (threads / 32) * N : 0)) * sizeof(float);
+    const int rows = N + (gate_out ? 1 : 0);
+    const size_t smem = (size_t)(2 * rows + n_groups + (vec ? (threads / 32) * rows : 0)) * sizeof(float);
     if (smem > 48 * 1024) return FWB_TOO_LARGE;
     if (h_bf16)
         fwb::pdl(moe_route_kernel<__nv_bfloat16>, blocks, threads, smem, stream)(
-            (const __nv_bfloat16*)h, router, correction, ids, weights, T, W, N, n_groups, keep, top, vec, scoring);
+            (const __nv_bfloat16*)h, router, correction, ids, weights, T, W, N, n_groups, keep, top, vec, scoring, gate_out);
     else
         fwb::pdl(moe_route_kernel<float>, blocks, threads, smem, stream)((const float*)h, router, correction, ids,
-                                                                          weights, T, W, N, n_groups, keep, top, vec, scoring);
+                                                                          weights, T, W, N, n_groups, keep, top, vec, scoring,
+                                                                          gate_out);
     return fwb_launch_status();
 }
 
-// The same choice from router outputs that are there already: logits fp32 [T][N].
+// The same choice from router outputs that are there already: logits fp32 [T][ld], ld >= N (+ 1 with gate_out).
 FWB_API int fwb_moe_choose(const float* logits, const float* correction, int* ids, float* weights, int T, int N,
-                           int n_groups, int keep, int top, int scoring, cudaStream_t stream) {
+                           int n_groups, int keep, int top, int scoring, long long ld, float* gate_out,
+                           cudaStream_t stream) {
     if (T <= 0) return FWB_OK;
-    if (!logits || !ids || !weights || scoring < 0 || scoring > 1) return FWB_BAD_ARGUMENT;
+    if (!logits || !ids || !weights || scoring < 0 || scoring > 2 || ld < N + (gate_out ? 1 : 0)) return FWB_BAD_ARGUMENT;
     if (N <= 0 || n_groups <= 0 || N % n_groups || keep <= 0 || keep > n_groups || top <= 0 || top > keep * (N / n_groups))
         return FWB_BAD_ARGUMENT;
     const size_t smem = (size_t)4 * (2 * N + n_groups) * sizeof(float);
     if (smem > 48 * 1024) return FWB_TOO_LARGE;
     fwb::pdl(moe_choose_kernel, (T + 3) / 4, 128, smem, stream)(logits, correction, ids, weights, T, N, n_groups, keep, top,
-                                                                scoring);
+                                                                scoring, ld, gate_out);
     return fwb_launch_status();
 }
 
@@ -651,14 +696,15 @@ FWB_API int fwb_moe_gather_rows(const void* h, const int* row_token, const int* 
 }
 
 // form 1: x [T][K] (rows gathered by row_token), w [E][2N][K], out [A][N] in the dtype of x.
+// form 2: x [T][K] (rows gathered by row_token), w [E][N][K], out [A][N] in the dtype of x, act an OUTPUT_* code.
 // form 0: x [A][K] sorted rows, w [E][N][K], out [A][N] fp32.
-// x and w are both fp32 or both bf16.  row_weight: [A] or null, multiplies the inputs of form 1.  max_tiles: the most tiles the sorted list can hold (the grid).
+// x and w are both fp32 or both bf16.  row_weight: [A] or null, multiplies the inputs of forms 1 and 2.  max_tiles: the most tiles the sorted list can hold (the grid).
 FWB_API int fwb_moe_gemm(const void* x, const void* w, int bf16, void* out, const int* offsets,
                          const int* row_token, const int* tiles, int max_tiles, int N, int K, int form, int act,
                          float limit, const float* row_weight, cudaStream_t stream) {
     if (max_tiles <= 0) return FWB_OK;
-    if (!x || !w || !out || !offsets || !row_token || !tiles || N <= 0 || K <= 0 || form < 0 || form > 1 ||
-        act < 0 || act > 2)
+    if (!x || !w || !out || !offsets || !row_token || !tiles || N <= 0 || K <= 0 || form < 0 || form > 2 ||
+        act < 0 || act > 3)
         return FWB_BAD_ARGUMENT;
     if (max_tiles > 65535) return FWB_TOO_LARGE;
     const dim3 grid((N + TN - 1) / TN, max_tiles);
@@ -669,6 +715,12 @@ FWB_API int fwb_moe_gemm(const void* x, const void* w, int bf16, void* out, cons
     else if (form == 1)
         fwb::pdl(moe_gemm_kernel<float, float, float, 1>, grid, 256, 0, stream)(
             (const float*)x, (const float*)w, (float*)out, offsets, row_token, tiles, N, K, act, limit, row_weight);
+    else if (form == 2 && bf16)
+        fwb::pdl(moe_gemm_kernel<bf, bf, bf, 2>, grid, 256, 0, stream)((const bf*)x, (const bf*)w, (bf*)out, offsets,
+                                                                       row_token, tiles, N, K, act, limit, row_weight);
+    else if (form == 2)
+        fwb::pdl(moe_gemm_kernel<float, float, float, 2>, grid, 256, 0, stream)(
+            (const float*)x, (const float*)w, (float*)out, offsets, row_token, tiles, N, K, act, limit, row_weight);
     else if (bf16)
         fwb::pdl(moe_gemm_kernel<bf, bf, float, 0>, grid, 256, 0, stream)((const bf*)x, (const bf*)w, (float*)out,
                                                                           offsets, row_token, tiles, N, K, act, limit, row_weight);
@@ -678,27 +730,31 @@ FWB_API int fwb_moe_gemm(const void* x, const void* w, int bf16, void* out, cons
     return fwb_launch_status();
 }
 
-// y: [A][W] fp32 sorted rows; h: [T][W]; out: [T][W] fp32.  weighted_in: the rows were weighted on their way in.
+// y: [A][W] fp32 sorted rows; h: [T][W]; out: [T][W] fp32.  extra, extra_gate: as in fwb_moe_combine_norm_add.
+// weighted_in: the rows were weighted on their way in.
 FWB_API int fwb_moe_combine(const float* y, const void* h, int h_bf16, const int* pair_row, const int* ids,
-                            const float* weights, float* out, int T, int W, int top, int E, int weighted_in,
+                            const float* weights, float* out, int T, int W, int top, int E, const float* extra,
+                            const float* extra_gate, int weighted_in,
                             cudaStream_t stream) {
     if (T <= 0) return FWB_OK;
     if (!y || !h || !pair_row || !ids || !weights || !out || W <= 0 || top <= 0) return FWB_BAD_ARGUMENT;
     if (top > 64) return FWB_TOO_LARGE;
     if (h_bf16)
         fwb::pdl(moe_combine_kernel<__nv_bfloat16>, T, 256, 0, stream)(y, (const __nv_bfloat16*)h, pair_row, ids,
-                                                                       weights, out, W, top, E, weighted_in);
+                                                                       weights, out, W, top, E, extra, extra_gate, weighted_in);
     else
         fwb::pdl(moe_combine_kernel<float>, T, 256, 0, stream)(y, (const float*)h, pair_row, ids, weights, out, W,
-                                                               top, E, weighted_in);
+                                                               top, E, extra, extra_gate, weighted_in);
     return fwb_launch_status();
 }
 
-// The same sum (plus row t of `extra`, fp32 [T][W] or null: what every token gets besides its experts), then
+// The same sum (plus row t of `extra`, fp32 [T][W] or null: what every token gets besides its experts; times
+// extra_gate[t] when that is given), then
 // x[t] += norm_w * sum / sqrt(mean(sum^2) + eps) in place (x: [T][W] fp32).
 FWB_API int fwb_moe_combine_norm_add(const float* y, const void* h, int h_bf16, const int* pair_row, const int* ids,
                                      const float* weights, float* x, const float* norm_w, float eps, int T, int W,
-                                     int top, int E, const float* extra, int weighted_in, cudaStream_t stream) {
+                                     int top, int E, const float* extra, const float* extra_gate, int weighted_in,
+                                     cudaStream_t stream) {
     if (T <= 0) return FWB_OK;
     if (!y || !h || !pair_row || !ids || !weights || !x || !norm_w || W <= 0 || top <= 0) return FWB_BAD_ARGUMENT;
     if (top > 64) return FWB_TOO_LARGE;
@@ -708,12 +764,13 @@ FWB_API int fwb_moe_combine_norm_add(const float* y, const void* h, int h_bf16, 
         if (smem > 48 * 1024)
             cudaFuncSetAttribute(moe_combine_norm_add_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         fwb::pdl(moe_combine_norm_add_kernel<__nv_bfloat16>, T, 256, smem, stream)(
-            y, (const __nv_bfloat16*)h, pair_row, ids, weights, x, norm_w, eps, W, top, E, extra, weighted_in);
+            y, (const __nv_bfloat16*)h, pair_row, ids, weights, x, norm_w, eps, W, top, E, extra, extra_gate,
+            weighted_in);
     } else {
         if (smem > 48 * 1024)
             cudaFuncSetAttribute(moe_combine_norm_add_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         fwb::pdl(moe_combine_norm_add_kernel<float>, T, 256, smem, stream)(y, (const float*)h, pair_row, ids, weights, x,
-                                                                           norm_w, eps, W, top, E, extra, weighted_in);
+                                                                           norm_w, eps, W, top, E, extra, extra_gate, weighted_in);
     }
     return fwb_launch_status();
 }

@@ -76,11 +76,11 @@ FWB_API int fwb_rmsnorm_add(float* x, const float* y, const float* w, float eps,
 }
 
 // gu: [T][2F] (gate columns, then up columns); out: [T][F].  act: 0 silu, 1 gelu (tanh form), 2 the clamped
-// swish with its `limit`.
+// swish with its `limit`, 3 relu.
 FWB_API int fwb_gate_act_mul(const void* gu, int in_bf16, void* out, int out_bf16, int T, int F, int act,
                              float limit, cudaStream_t stream) {
     if (T <= 0) return FWB_OK;
-    if (!gu || !out || F <= 0 || act < 0 || act > 2) return FWB_BAD_ARGUMENT;
+    if (!gu || !out || F <= 0 || act < 0 || act > 3) return FWB_BAD_ARGUMENT;
     const size_t n = (size_t)T * F;
     const int blocks = (int)((n + 255) / 256 > 8192 ? 8192 : (n + 255) / 256);
     if (in_bf16 && out_bf16)

@@ -223,14 +223,15 @@ __device__ __forceinline__ float gate_act_fast(int act, float g) {
     return __fdividef(g, 1.0f + __expf(-z));
 }
 // The gated value of the epilogue, act(g) * u; 2 = the clamped swish (g cut off above `limit`, u held inside
-// [-limit, limit], g sigmoid(1.702 g) (u + 1)), the same quotient once more.
-constexpr int GATE_SWISH_CLAMPED = 2;
+// [-limit, limit], g sigmoid(1.702 g) (u + 1)), the same quotient once more; 3 = max(g, 0) u.
+constexpr int GATE_SWISH_CLAMPED = 2, GATE_RELU = 3;
 __device__ __forceinline__ float gated_fast(int act, float limit, float g, float u) {
     if (act == GATE_SWISH_CLAMPED) {
         g = fminf(g, limit);
         u = fminf(fmaxf(u, -limit), limit) + 1.0f;
         return __fdividef(g, 1.0f + __expf(-1.702f * g)) * u;
     }
+    if (act == GATE_RELU) return fmaxf(g, 0.0f) * u;
     return gate_act_fast(act, g) * u;
 }
 

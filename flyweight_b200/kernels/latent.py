@@ -100,6 +100,35 @@ def latent_prepare(proj: torch.Tensor, kv_col: int, norm_w: Optional[torch.Tenso
     return qa
 
 
+def latent_low_rank(proj: torch.Tensor, q_rank: int, q_norm_w: torch.Tensor, norm_w: Optional[torch.Tensor],
+                    table: torch.Tensor, batch, block_table: Optional[torch.Tensor], pool: Optional[torch.Tensor],
+                    rot: int, rot_dims: int, pairing: str, rank: int, row: int, eps: float,
+                    out_dtype: torch.dtype) -> torch.Tensor:
+    """From rows ``proj`` = [queries' row (q_rank) | latent (rank) | shared key part (rot)]: the queries' row,
+    RMS-normed and weighted, [T][q_rank] in ``out_dtype``; and (with ``pool``) the token's cache row as
+    ``latent_prepare`` writes it."""
+    check_tensor("low-rank projection", proj)
+    check_tensor("query latent norm weight", q_norm_w, torch.float32, (q_rank,))
+    T, ld = proj.shape
+    page_size = max_pages = 0
+    if pool is not None:
+        check_tensor("rope table", table, torch.float32)
+        if table.dim() != 3 or table.shape[1] != max(1, rot_dims // 2) or table.shape[2] != 2:
+            raise KernelError("rope table must be [positions][rot_dims/2][2]")
+        check_tensor("latent pool", pool)
+        check_tensor("latent norm weight", norm_w, torch.float32, (rank,))
+        _i32("block table", block_table)
+        if pool.dim() != 4 or pool.shape[1] != 1 or pool.shape[3] != row:
+            raise KernelError(f"the latent pool must be [pages][1][page_size][{row}], got {tuple(pool.shape)}")
+        page_size, max_pages = pool.shape[2], block_table.shape[1]
+    cq = torch.empty((T, q_rank), dtype=out_dtype, device=proj.device)
+    lib.call("fwb_latent_low_rank", ptr(proj), is_bf16(proj), ld, int(q_rank), ptr(q_norm_w), ptr(norm_w), ptr(table),
+             ptr(batch.positions), ptr(batch.tok_seg), ptr(block_table), max_pages, page_size, ptr(cq), is_bf16(cq),
+             ptr(pool), is_bf16(pool) if pool is not None else 0, T, rot, rot_dims, ROPE_PAIRINGS[pairing], rank, row,
+             c_float(eps), stream())
+    return cq
+
+
 _mma_enabled = True
 
 

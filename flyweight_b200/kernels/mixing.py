@@ -44,18 +44,23 @@ def rmsnorm_ranges_(buf: torch.Tensor, ranges) -> torch.Tensor:
 
 
 def causal_conv(rows: torch.Tensor, taps: torch.Tensor, state: Optional[torch.Tensor], batch,
-                norm_ranges=None) -> torch.Tensor:
-    """A causal convolution over time on the first C channels of ``rows`` ([T][>= C], fp32 or bf16), ``taps`` fp32
+                norm_ranges=None, col0: int = 0, bias: Optional[torch.Tensor] = None, silu: bool = False,
+                out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+    """A causal convolution over time on C channels of ``rows`` ([T][>= col0 + C], fp32 or bf16) from column
+    ``col0`` on, ``taps`` fp32
     [C][n] with the last tap on the token itself: ``y[t] = sum_j taps[:, j] * rows[t - n + 1 + j]`` along each
     request's tokens.  ``state``: fp32 [slots][n - 1][C], every live request's last n - 1 inputs (zero when it
     starts), read in front of a portion and moved on by this call (None when n == 1).  ``norm_ranges``: one or two
     ``(col0, weight, count, eps)`` as ``rmsnorm_ranges_`` takes them; those column ranges of the result are
-    normed by the same launch.  Returns a new buffer [T][C]; ``rows`` (and its columns from C on) stay."""
+    normed by the same launch.  ``bias``: fp32 [C], added to the convolved value; ``silu``: which then passes silu.
+    Returns a new buffer [T][C] in ``out_dtype`` (that of ``rows`` when None); ``rows`` stays."""
     check_tensor("convolution input", rows)
     T, ld = rows.shape
     C, n = taps.shape
     check_tensor("convolution taps", taps, torch.float32)
-    if C > ld:
+    if bias is not None:
+        check_tensor("convolution bias", bias, torch.float32, (C,))
+    if col0 < 0 or col0 + C > ld:
         raise KernelError(f"taps for {C} channels, rows of {ld}")
     stride = 0
     if n > 1:
@@ -74,8 +79,9 @@ def causal_conv(rows: torch.Tensor, taps: torch.Tensor, state: Optional[torch.Te
             if float(this_eps) != eps:
                 raise KernelError("the ranges of one launch share their eps")
             norm_args[4 * index:4 * index + 4] = [int(col0), weight.numel(), int(count), ptr(weight)]
-    out = torch.empty((T, C), dtype=rows.dtype, device=rows.device)
-    lib.call("fwb_causal_conv", ptr(rows), ptr(out), is_bf16(rows), c_longlong(ld), c_longlong(C), 0, C, ptr(taps), n,
+    out = torch.empty((T, C), dtype=out_dtype or rows.dtype, device=rows.device)
+    lib.call("fwb_causal_conv", ptr(rows), ptr(out), is_bf16(rows), is_bf16(out), ptr(bias), 1 if silu else 0,
+             c_longlong(ld), c_longlong(C), int(col0), C, ptr(taps), n,
              ptr(state) if n > 1 else None, c_longlong(stride), ptr(batch.tok_seg), ptr(batch.seg_start),
              ptr(batch.seg_slot), T, batch.n_segments, *norm_args, c_float(eps), stream(),
              launches=2 if n > 1 else 1)

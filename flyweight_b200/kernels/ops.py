@@ -168,6 +168,17 @@ def linear(x, w: torch.Tensor, out_dtype: torch.dtype,
     return gemm_simt(x, w, out_dtype, addend)
 
 
+def linear_act(x: torch.Tensor, w: torch.Tensor, activation: str, out_dtype: torch.dtype) -> torch.Tensor:
+    """``act(x @ w.T)``, the activation (one of ``OUTPUT_ACTIVATIONS``) on the product's fp32 sums: in the tensor-core
+    product's epilogue when the output is bfloat16, else as a pass of its own."""
+    from . import mixing, tensorcore
+    if w.dtype == torch.bfloat16 and out_dtype == torch.bfloat16:
+        x = cast(x, torch.bfloat16)
+        if tensorcore.accepts(x, w, out_dtype):
+            return tensorcore.gemm(x, w, out_dtype, activation=activation)
+    return mixing.unary_act(linear(x, w, torch.float32), activation, out_dtype)
+
+
 def linear_into_residual(x: torch.Tensor, w: torch.Tensor, residual: Optional[torch.Tensor]):
     """``residual += x @ w.T`` in the product's epilogue when the tensor-core kernel has that
     form for the shape (returns None); otherwise the fp32 product, for the caller to hand on."""
@@ -192,14 +203,16 @@ def silu_mul(gate_up: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
 
 
 # what a gated feed-forward makes of gate g and up u: silu(g) u, gelu(g) u (tanh form), or the clamped swish
-# min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1) with a limit L
-GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "swish_clamped": 2}
+# min(g, L) sigmoid(1.702 min(g, L)) (clamp(u, -L, L) + 1) with a limit L, or max(g, 0) u
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "swish_clamped": 2, "relu": 3}
+# what a product without a gate may do to a bfloat16 output on its way out (in fp32, ahead of the rounding)
+OUTPUT_ACTIVATIONS = {None: 0, "relu_squared": 1}
 
 
 def gate_act_mul(gate_up: torch.Tensor, out_dtype: torch.dtype, activation: str = "silu",
                  limit: float = 0.0) -> torch.Tensor:
     """``act(gate) * up`` for ``gate_up`` = [T][gate(F) | up(F)]; ``activation``: "silu", "gelu_tanh"
-    (0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3)))) or "swish_clamped" with its ``limit``."""
+    (0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3)))), "swish_clamped" with its ``limit``, or "relu"."""
     check_tensor("gate|up", gate_up)
     T, F2 = gate_up.shape
     if F2 % 2:

@@ -19,6 +19,13 @@ def _gated_epilogue(activation: str) -> int:
     from .ops import GATE_ACTIVATIONS
     return EPI_SWIGLU_BF16 | (GATE_ACTIVATIONS[activation] << GATE_ACT_SHIFT)
 
+
+def _output_epilogue(activation) -> int:
+    """A bfloat16 output with an activation of ``ops.OUTPUT_ACTIVATIONS`` applied in fp32 in front of the rounding."""
+    from .ops import OUTPUT_ACTIVATIONS
+    return EPI_BF16 | (OUTPUT_ACTIVATIONS[activation] << GATE_ACT_SHIFT)
+
+
 SM_COUNT = 148
 _enabled = True
 
@@ -190,9 +197,11 @@ def adds_in_place(x, w, residual) -> bool:
             and tuple(residual.shape) == (x.shape[0], w.shape[0]))
 
 
-def gemm(x, w, out_dtype, addend=None, splits=None, stages=0, tile_tokens=0, wide=-1, out=None) -> torch.Tensor:
+def gemm(x, w, out_dtype, addend=None, splits=None, stages=0, tile_tokens=0, wide=-1, out=None,
+         activation=None) -> torch.Tensor:
     """``x @ w.T``: x [M][K] bf16, w [N][K] bf16 -> [M][N] fp32 or bf16 (+ fp32 addend).
-    ``out`` may be the addend itself (the sum in place)."""
+    ``out`` may be the addend itself (the sum in place).  ``activation`` (bf16 outputs): one of
+    ``ops.OUTPUT_ACTIVATIONS``, applied on the way out."""
     check_tensor("gemm input", x, torch.bfloat16)
     check_tensor("gemm weight", w, torch.bfloat16)
     M, K = x.shape
@@ -200,16 +209,18 @@ def gemm(x, w, out_dtype, addend=None, splits=None, stages=0, tile_tokens=0, wid
     if w.shape[1] != K:
         raise KernelError(f"gemm: input has {K} columns, weight has {w.shape[1]}")
     free_choice = splits is None and not stages and not tile_tokens and wide == -1
+    if activation is not None and (out_dtype != torch.bfloat16 or addend is not None):
+        raise KernelError("an activation on the way out goes with a bfloat16 output")
     pair_ok = _use_pairs and M > 128 and addend is None and out is None and N >= 256
     if free_choice and _mid_size_split and MID_FROM <= M <= MID_TO:
         kind, tile_tokens, splits = mid_size_choice(M, N, K, 1, pair_ok)
         if kind == "pair":
-            return gemm_pair(x, w, out_dtype, wide=False)
+            return gemm_pair(x, w, out_dtype, wide=False, activation=activation)
     elif pair_ok and free_choice:
         # prompt-sized: CTA pairs (cta_group::2); two feature blocks per pair when single blocks
         # would make more CTAs than the GPU holds at once (measured at 2,048 tokens on B200)
         pairs = -(-N // 256) * -(-M // 256)
-        return gemm_pair(x, w, out_dtype, wide=pairs > SM_COUNT // 2)
+        return gemm_pair(x, w, out_dtype, wide=pairs > SM_COUNT // 2, activation=activation)
     if out is None:
         out = torch.empty((M, N), dtype=out_dtype, device=x.device)
     else:
@@ -218,7 +229,7 @@ def gemm(x, w, out_dtype, addend=None, splits=None, stages=0, tile_tokens=0, wid
         check_tensor("gemm addend", addend, torch.float32, (M, N))
         epilogue = EPI_ADD_F32
     else:
-        epilogue = EPI_F32 if out_dtype == torch.float32 else EPI_BF16
+        epilogue = EPI_F32 if out_dtype == torch.float32 else _output_epilogue(activation)
     if M <= 64 and (N, K, 1) in TUNED and _forced_splits is None:
         tuned = TUNED[(N, K, 1)]
         splits = splits or tuned[0] or None
@@ -400,7 +411,7 @@ def status() -> int:
     return int(lib.library().fwb_gemm_tcgen05_status())
 
 
-def gemm_pair(x, w, out_dtype, wide=False) -> torch.Tensor:
+def gemm_pair(x, w, out_dtype, wide=False, activation=None) -> torch.Tensor:
     """``x @ w.T`` on CTA pairs (tcgen05 cta_group::2): 256 features x 256 tokens per pair and
     accumulator.  For prompt-sized steps; bf16 in, fp32 or bf16 out."""
     check_tensor("gemm input", x, torch.bfloat16)
@@ -410,7 +421,7 @@ def gemm_pair(x, w, out_dtype, wide=False) -> torch.Tensor:
     if w.shape[1] != K:
         raise KernelError(f"gemm: input has {K} columns, weight has {w.shape[1]}")
     out = torch.empty((M, N), dtype=out_dtype, device=x.device)
-    epilogue = EPI_F32 if out_dtype == torch.float32 else EPI_BF16
+    epilogue = EPI_F32 if out_dtype == torch.float32 else _output_epilogue(activation)
     cut = _pair_wave_cut(M, N) if wide else 0
     if cut:
         # the wide blocks of the whole rounds, then the rest as narrow pairs that fit one round

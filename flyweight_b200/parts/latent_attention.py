@@ -42,7 +42,9 @@ class LatentAttention(Mixer):
     whose ``rotary_dim`` <= rot_dim), sink (True: a learned number per head joins the softmax
     denominator), shares_cache (True: reads the rows of another execution; no latent projection), gate
     ("head": tensor ``g`` [heads][H], every head's output times sigmoid(g h) of its head, from the mixer's
-    own input).  tensors: q, dkv, dkv_norm, uk, uv, o, sink, g."""
+    own input), q_rank (> 0: the queries come from a
+    low-rank row that is RMS-normed with a weight in between, q = W_uq (w * unit(W_dq h)); tensors dq [q_rank][H],
+    dq_norm [q_rank], uq instead of q).  tensors: q, dkv, dkv_norm, uk, uv, o, sink, g."""
     graph_safe = True
 
     def __init__(self, spec):
@@ -61,6 +63,9 @@ class LatentAttention(Mixer):
         self.gate = p.get("gate")
         if self.gate not in (None, "head"):
             raise ValueError(f"unknown output gate {self.gate!r}; known: head")
+        self.q_rank = int(p.get("q_rank", 0) or 0)
+        if self.q_rank and self.gate:
+            raise ValueError("an output gate and queries from a low-rank row have no form together")
         self.position = build_position(p["position"])
         if self.position.rotary_dim > self.rot:
             raise ValueError(f"{self.position.rotary_dim} turning channels but a rotated part of {self.rot}")
@@ -72,13 +77,19 @@ class LatentAttention(Mixer):
         self.row = 64 if used <= 64 else (128 if 96 < used <= 128 else _round_up(used, 16))
         self.q_width = self.n_heads * (self.dim + self.rot)
         self.w_in = self.w_uk_t = self.w_uv = self.w_o = self.norm_w = self.sink = self.w_gate = None
+        self.w_uq = self.q_norm_w = None
 
     def declare(self):
         n, H = self.names, self.hidden
-        out = {n["q"]: TensorDecl((self.q_width, H)),
-               n["uk"]: TensorDecl((self.n_heads * self.dim, self.rank)),
+        out = {n["uk"]: TensorDecl((self.n_heads * self.dim, self.rank)),
                n["uv"]: TensorDecl((self.n_heads * self.vdim, self.rank)),
                n["o"]: TensorDecl((H, self.n_heads * self.vdim))}
+        if self.q_rank:
+            out[n["dq"]] = TensorDecl((self.q_rank, H))
+            out[n["dq_norm"]] = TensorDecl((self.q_rank,), "norm")
+            out[n["uq"]] = TensorDecl((self.q_width, self.q_rank))
+        else:
+            out[n["q"]] = TensorDecl((self.q_width, H))
         if not self.shares_cache:
             out[n["dkv"]] = TensorDecl((self.rank + self.rot, H))
             out[n["dkv_norm"]] = TensorDecl((self.rank,), "norm")
@@ -90,7 +101,7 @@ class LatentAttention(Mixer):
 
     def bind(self, get, precision: Precision, device):
         n = self.names
-        mats = [get(n["q"])] + ([] if self.shares_cache else [get(n["dkv"])])
+        mats = [get(n["dq" if self.q_rank else "q"])] + ([] if self.shares_cache else [get(n["dkv"])])
         self._gate_col = sum(m.shape[0] for m in mats)
         if self.gate:
             gate_rows = get(n["g"])
@@ -105,13 +116,16 @@ class LatentAttention(Mixer):
         self.w_uk_t = precision.matrix(uk.contiguous(), device)
         self.w_uv = precision.matrix(get(n["uv"]).reshape(self.n_heads, self.vdim, self.rank), device)
         self.w_o = precision.matrix(get(n["o"]), device)
+        if self.q_rank:
+            self.w_uq = precision.matrix(get(n["uq"]), device)
+            self.q_norm_w = precision.vector(get(n["dq_norm"]), device)
         if not self.shares_cache:
             self.norm_w = precision.vector(get(n["dkv_norm"]), device)
         if self.has_sink:
             self.sink = precision.vector(get(n["sink"]), device)
 
     def _matrices(self):
-        return tuple(m for m in (self.w_in, self.w_uk_t, self.w_uv, self.w_o, self.w_gate) if m is not None)
+        return tuple(m for m in (self.w_in, self.w_uq, self.w_uk_t, self.w_uv, self.w_o, self.w_gate) if m is not None)
 
     def weight_bytes(self):
         return sum(m.numel() * m.element_size() for m in self._matrices())
@@ -136,6 +150,8 @@ class LatentAttention(Mixer):
         rotation = self.position.rotation()
         if rotation is None:
             raise NotPlannable(f"position encoding {self.position.kind!r} is no plain rotation")
+        if self.q_rank:
+            raise NotPlannable("queries from a low-rank row have no native plan form")
         if self.gate:
             raise NotPlannable("an output gate on the latent attention has no native plan form")
         table, rot_dims, pairing = rotation
@@ -163,10 +179,18 @@ class LatentAttention(Mixer):
                              f"{self.position.kind!r} is no plain rotation")
         table, rot_dims, pairing = rotation
         block_table = batch.block_tables[cache.group]
-        proj = ops.linear(h, self.w_in, act)                     # [T][queries | latent + key part]
+        pool = None if self.shares_cache else cache.k_pool
+        if self.q_rank:
+            # [T][queries' row | latent + key part] stays in fp32 up to its two norms
+            cq = latent_kernels.latent_low_rank(
+                ops.linear(h, self.w_in, torch.float32), self.q_rank, self.q_norm_w, self.norm_w, table, batch,
+                block_table, pool, self.rot, rot_dims, pairing, self.rank, self.row, self.eps, act)
+            proj, pool = ops.linear(cq, self.w_uq, act), None    # the cache row is written
+        else:
+            proj = ops.linear(h, self.w_in, act)                 # [T][queries | latent + key part]
         qa = latent_kernels.latent_prepare(
             proj, self.q_width, self.norm_w, table, batch, block_table,
-            None if self.shares_cache else cache.k_pool, self.n_heads, self.dim, self.rot, rot_dims, pairing,
+            pool, self.n_heads, self.dim, self.rot, rot_dims, pairing,
             self.rank, self.row, self.eps)
         qa2 = qa.view(qa.shape[0], self.n_heads * self.row)
         latent_kernels.head_linear(proj, 0, self.dim + self.rot, self.dim, self.w_uk_t, qa2, 0, self.row)
