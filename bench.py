@@ -165,6 +165,35 @@ def vugipel_like(lfm2: dict, ff: int) -> dict:
             "layers": layers}
 
 
+def futezen_like(lfm2: dict, ff: int) -> dict:
+    """A Futezen configuration with the layer sizes of an LFM2 one (width, vocabulary, query and key/value heads of
+    64; as many layer executions as LFM2 has layers: two layers fewer, with layers 2 and 3 run twice).  Where LFM2
+    attends, grouped-query attention and attention over a cached latent in turn (64 plain and 32 turned query channels
+    a head from a low-rank row of 3/8 of the width, a latent of 256: a cache row of 288), with a dense feed-forward;
+    where it has a short convolution, a state-space recurrence of twice the width (heads of 64 channels, 128 state
+    rows, one group, 4 taps) with 16 experts of ff / 8, four a token, beside a shared expert of ff / 2."""
+    width, heads, kv = lfm2["hidden_size"], lfm2["num_attention_heads"], lfm2["num_key_value_heads"]
+    experts = {"kind": "moe", "expert": {"ff": ff // 8}, "router": {"experts": 16, "top": 4}, "shared": {"ff": ff // 2}}
+    dense = {"kind": "dense", "ff": ff}
+    layers, attending = [], 0
+    for index in range(lfm2["num_hidden_layers"] - 2):
+        if index not in lfm2["full_attn_idxs"]:
+            mixer = {"heads": 2 * width // 64, "vdim": 64, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
+            layers.append({"type": "mamba2", "mixer": mixer, "mlp": experts})
+            continue
+        if attending % 2 == 0:
+            mixer = {"heads": heads, "dim": 64, "rot_dim": 32, "vdim": 64, "q_rank": 3 * width // 8, "kv_rank": 256,
+                     "scale": 96 ** -0.5, "rot": {"base": 10000.0, "dims": 32}}
+            layers.append({"type": "latent_attention", "mixer": mixer, "mlp": dense})
+        else:
+            mixer = {"heads": heads, "kv_heads": kv, "dim": 64, "vdim": 64, "scale": 0.125,
+                     "rot": {"base": 1000000.0, "dims": 64}}
+            layers.append({"type": "attention", "mixer": mixer, "mlp": dense})
+        attending += 1
+    return {"architecture": "Futezen", "vocab": lfm2["vocab_size"], "width": width, "norm": {"eps": 1e-5},
+            "loop": {"start": 2, "stop": 4, "times": 2}, "layers": layers}
+
+
 # Kemitar, Diforax and Gukosun beside LFM2 at equal layer sizes (--compare): the feed-forward widths are what
 # LFM2's rule makes of ``intermediate_size`` at these sizes.
 KEMITAR = {"kemitar-350m": ("lfm2-350m", 4608), "kemitar-1.2b": ("lfm2-1.2b", 8192)}
@@ -186,7 +215,12 @@ for _name, (_twin, _ff) in FOBATAR.items():
 VUGIPEL = {"vugipel-350m": ("gukosun-350m", 4608), "vugipel-1.2b": ("gukosun-1.2b", 8192)}
 for _name, (_twin, _ff) in VUGIPEL.items():
     MODELS[_name] = vugipel_like(MODELS["lfm2" + _name[len("vugipel"):]], _ff)
-COMPARE = {**KEMITAR, **DIFORAX, **GUKOSUN, **FOBATAR, **VUGIPEL}
+# Futezen beside Fobatar, the closest model the engine has (a norm on both sides of every sublayer, attention over
+# a cached latent, experts beside a shared one, repeated layers), at equal layer sizes
+FUTEZEN = {"futezen-350m": ("fobatar-350m", 4608), "futezen-1.2b": ("fobatar-1.2b", 8192)}
+for _name, (_twin, _ff) in FUTEZEN.items():
+    MODELS[_name] = futezen_like(MODELS["lfm2" + _name[len("futezen"):]], _ff)
+COMPARE = {**KEMITAR, **DIFORAX, **GUKOSUN, **FOBATAR, **VUGIPEL, **FUTEZEN}
 
 
 def vocab_of(config: dict) -> int:
@@ -581,8 +615,8 @@ def run_sizes(args) -> int:
 
 def run_compare(args) -> int:
     """``--compare kemitar-350m|kemitar-1.2b|diforax-350m|diforax-1.2b|gukosun-350m|gukosun-1.2b|fobatar-350m|fobatar-1.2b|
-    vugipel-350m|vugipel-1.2b``: the model with random weights beside its twin (LFM2; for Fobatar, Diforax; for
-    Vugipel, Gukosun) at equal layer sizes, both through the same step function -- prompts of 512, 2,048 and 8,192 tokens in one step
+    vugipel-350m|vugipel-1.2b|futezen-350m|futezen-1.2b``: the model with random weights beside its twin (LFM2; for
+    Fobatar, Diforax; for Vugipel, Gukosun; for Futezen, Fobatar) at equal layer sizes, both through the same step function -- prompts of 512, 2,048 and 8,192 tokens in one step
     (tokens/s and TFLOP/s of the model's own flop count) and decode steps at batch 1, 8 and 64 over 4,096
     cached tokens (tokens/s, and the bytes a step must read against the measured copy bandwidth).  One
     JSON line per model; the LFM2 line's ffn width is checked to be the one the Kemitar twin was given."""
@@ -911,7 +945,7 @@ def main() -> int:
                              "requests, 256 new tokens each, through the public runtime (e.g. lfm2-350m)")
     parser.add_argument("--compare", default=None, metavar="MODEL",
                         help="kemitar-350m, kemitar-1.2b, diforax-350m, diforax-1.2b, gukosun-350m or gukosun-1.2b beside LFM2, "
-                             "fobatar-350m or fobatar-1.2b beside Diforax, vugipel-350m or vugipel-1.2b beside Gukosun, at equal layer sizes: prompts and decode steps")
+                             "fobatar-350m or fobatar-1.2b beside Diforax, vugipel-350m or vugipel-1.2b beside Gukosun, futezen-350m or futezen-1.2b beside Fobatar, at equal layer sizes: prompts and decode steps")
     parser.add_argument("--kernel-times", default=None, metavar="[MODEL:]decode[@BATCHxCONTEXT]|prefill|TOKENS",
                         help="one step with CUDA events around every launch: time per kernel as JSON")
     args = parser.parse_args()

@@ -76,6 +76,7 @@ struct AttnParams {
     const int* tile_tok0;        // [n_tiles]
     const int* block_table;      // [S][max_pages]
     int max_pages, nh, nkv, group, tokens_per_tile, window, n_row_tiles;
+    int head_cols;               // 1: keys and values are token-major rows, a head's channels side by side
     int items_per_cta;           // 2: CTA c takes items c and n-1-c; 1: one item each (few items)
     float scale_log2;            // softmax scale * log2(e)
     const float* sink;           // [nh] or null: a score per head (not scaled) in the softmax denominator, no value
@@ -205,6 +206,7 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
             bool ok = true;
             for (int it = 0; it < n_local && ok; ++it) {
                 const Item item = load_item(prm, it == 0 ? (int)blockIdx.x : second_item);
+                const int x0 = prm.head_cols ? item.kvh * HD : 0;
                 for (int t = 0; t < item.n_tiles + LEAD; ++t, ++u) {
                     const int s = u % L::STAGES;
                     if (u >= L::STAGES) ok = mbar_wait(&empty[s], ((u / L::STAGES) - 1) & 1, abort_flag, 11, prm.status);
@@ -212,16 +214,18 @@ attention_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k,
                     const bool has_k = t < item.n_tiles, has_v = t >= LEAD;
                     mbar_expect_tx(&full[s], ((has_k ? 1 : 0) + (has_v ? 1 : 0)) * L::KV_BYTES);
                     if (has_k) {
-                        const int row = (item.table[item.walk.at(t)] * prm.nkv + item.kvh) * KEYS;
+                        const int page = item.table[item.walk.at(t)];
+                        const int row = prm.head_cols ? page * KEYS : (page * prm.nkv + item.kvh) * KEYS;
 #pragma unroll
                         for (int b = 0; b < L::BOXES; ++b)
-                            tma_load_2d(k_s + (size_t)s * L::KV_BYTES + b * L::KV_BOX, &map_k, &full[s], b * 64, row);
+                            tma_load_2d(k_s + (size_t)s * L::KV_BYTES + b * L::KV_BOX, &map_k, &full[s], x0 + b * 64, row);
                     }
                     if (has_v) {
-                        const int row = (item.table[item.walk.at(t - LEAD)] * prm.nkv + item.kvh) * KEYS;
+                        const int page = item.table[item.walk.at(t - LEAD)];
+                        const int row = prm.head_cols ? page * KEYS : (page * prm.nkv + item.kvh) * KEYS;
 #pragma unroll
                         for (int b = 0; b < L::BOXES; ++b)
-                            tma_load_2d(v_s + (size_t)s * L::KV_BYTES + b * L::KV_BOX, &map_v, &full[s], b * 64, row);
+                            tma_load_2d(v_s + (size_t)s * L::KV_BYTES + b * L::KV_BOX, &map_v, &full[s], x0 + b * 64, row);
                     }
                 }
             }
@@ -526,6 +530,42 @@ FWB_API int fwb_attention_prefill_tcgen05_sink(const void* q, const void* k_pool
                                                 hd, tokens_per_tile, window, scale, sink, 0.0f, 0, stream);
 }
 
+namespace {
+int prefill_tcgen05(const void* q, const CUtensorMap& map_k, const CUtensorMap& map_v, int head_cols,
+                    const int* positions, const int* seg_start, const int* tile_seg, const int* tile_tok0,
+                    const int* block_table, int max_pages, void* out, int n_tiles, int nh, int nkv, int hd,
+                    int tokens_per_tile, int window, float scale, const float* sink, float softcap, int keep,
+                    cudaStream_t stream) {
+    AttnParams prm;
+    prm.q = static_cast<const __nv_bfloat16*>(q);
+    prm.out = static_cast<__nv_bfloat16*>(out);
+    prm.positions = positions;
+    prm.seg_start = seg_start;
+    prm.tile_seg = tile_seg;
+    prm.tile_tok0 = tile_tok0;
+    prm.block_table = block_table;
+    prm.max_pages = max_pages;
+    prm.nh = nh;
+    prm.nkv = nkv;
+    prm.group = nh / nkv;
+    prm.tokens_per_tile = tokens_per_tile;
+    prm.window = window;
+    prm.n_row_tiles = n_tiles;
+    prm.head_cols = head_cols;
+    // one CTA per SM is resident (the tiles fill shared memory): pairs of items even out the causal
+    // triangle when there are waves of them; up to one wave of single items, single items finish sooner
+    prm.items_per_cta = (long)n_tiles * nkv <= 148 ? 1 : 2;
+    prm.scale_log2 = scale * LOG2E;
+    prm.sink = sink;
+    prm.keep = keep;
+    prm.cap_pre = softcap > 0.0f ? scale / softcap : 0.0f;
+    prm.cap_unit = softcap > 0.0f ? softcap / scale : 0.0f;
+    prm.status = status_word();
+    return hd == 64 ? launch<64>(map_k, map_v, prm, n_tiles, stream)
+                    : launch<128>(map_k, map_v, prm, n_tiles, stream);
+}
+}  // namespace
+
 // The general form.  softcap > 0: score <- softcap * tanh(score / softcap) behind the scale (the sink is
 // not capped); a scale of 0 with a cap is refused (every score would be 0: not worth a form of its own).
 // keep > 0 (with a sliding window): the first `keep` positions stay visible beside the window.
@@ -550,30 +590,31 @@ FWB_API int fwb_attention_prefill_tcgen05_capped(const void* q, const void* k_po
     CUtensorMap map_k, map_v;
     if (!make_map(&map_k, k_pool, pool_rows, hd, KEYS)) return FWB_UNSUPPORTED;
     if (!make_map(&map_v, v_pool, pool_rows, hd, KEYS)) return FWB_UNSUPPORTED;
-    AttnParams prm;
-    prm.q = static_cast<const __nv_bfloat16*>(q);
-    prm.out = static_cast<__nv_bfloat16*>(out);
-    prm.positions = positions;
-    prm.seg_start = seg_start;
-    prm.tile_seg = tile_seg;
-    prm.tile_tok0 = tile_tok0;
-    prm.block_table = block_table;
-    prm.max_pages = max_pages;
-    prm.nh = nh;
-    prm.nkv = nkv;
-    prm.group = group;
-    prm.tokens_per_tile = tokens_per_tile;
-    prm.window = window;
-    prm.n_row_tiles = n_tiles;
-    // one CTA per SM is resident (the tiles fill shared memory): pairs of items even out the causal
-    // triangle when there are waves of them; up to one wave of single items, single items finish sooner
-    prm.items_per_cta = (long)n_tiles * nkv <= 148 ? 1 : 2;
-    prm.scale_log2 = scale * LOG2E;
-    prm.sink = sink;
-    prm.keep = keep;
-    prm.cap_pre = softcap > 0.0f ? scale / softcap : 0.0f;
-    prm.cap_unit = softcap > 0.0f ? softcap / scale : 0.0f;
-    prm.status = status_word();
-    return hd == 64 ? launch<64>(map_k, map_v, prm, n_tiles, stream)
-                    : launch<128>(map_k, map_v, prm, n_tiles, stream);
+    return prefill_tcgen05(q, map_k, map_v, 0, positions, seg_start, tile_seg, tile_tok0, block_table, max_pages, out,
+                           n_tiles, nh, nkv, hd, tokens_per_tile, window, scale, sink, softcap, keep, stream);
+}
+
+// Keys and values that are no pages but rows of a token-major buffer, head by head: k_rows, v_rows [n_rows][nh * hd],
+// rows `row_stride` entries apart (both may be columns of one buffer).  The block table names runs of 64 rows; every
+// head reads its own columns (no groups).
+FWB_API int fwb_attention_prefill_tcgen05_rows(const void* q, const void* k_rows, const void* v_rows,
+                                               long long row_stride, int n_rows, const int* positions,
+                                               const int* seg_start, const int* tile_seg, const int* tile_tok0,
+                                               const int* block_table, int max_pages, void* out, int n_tiles, int nh,
+                                               int hd, int tokens_per_tile, float scale, const float* sink,
+                                               cudaStream_t stream) {
+    if (n_tiles <= 0) return FWB_OK;
+    if (!q || !k_rows || !v_rows || !positions || !seg_start || !tile_seg || !tile_tok0 || !block_table || !out)
+        return FWB_BAD_ARGUMENT;
+    if (!fwb_attention_prefill_tcgen05_accepts(nh, nh, hd, KEYS)) return FWB_UNSUPPORTED;
+    if (tokens_per_tile < 1 || tokens_per_tile > ROWS || n_rows < KEYS || n_rows % KEYS || row_stride < (long long)nh * hd)
+        return FWB_BAD_ARGUMENT;
+    if ((((uintptr_t)q | (uintptr_t)out | (uintptr_t)k_rows | (uintptr_t)v_rows) & 15) != 0 || (row_stride & 7))
+        return FWB_UNSUPPORTED;
+    if ((long)n_tiles * nh > 2147483647L) return FWB_TOO_LARGE;
+    CUtensorMap map_k, map_v;
+    if (!make_map_strided(&map_k, k_rows, n_rows, nh * hd, row_stride, KEYS)) return FWB_UNSUPPORTED;
+    if (!make_map_strided(&map_v, v_rows, n_rows, nh * hd, row_stride, KEYS)) return FWB_UNSUPPORTED;
+    return prefill_tcgen05(q, map_k, map_v, 1, positions, seg_start, tile_seg, tile_tok0, block_table, max_pages, out,
+                           n_tiles, nh, nh, hd, tokens_per_tile, 0, scale, sink, 0.0f, 0, stream);
 }

@@ -286,16 +286,19 @@ inline EncodeTiledFn encode_fn() {
 }
 
 // A [rows][K] bf16 row-major matrix seen as boxes of [box_rows][64] with 128-byte swizzle.
-inline bool make_map(CUtensorMap* map, const void* base, long rows, int K, int box_rows) {
+inline bool make_map_strided(CUtensorMap* map, const void* base, long rows, int K, long row_stride, int box_rows) {
     EncodeTiledFn fn = encode_fn();
     if (!fn) return false;
     cuuint64_t dims[2] = {(cuuint64_t)K, (cuuint64_t)rows};
-    cuuint64_t strides[1] = {(cuuint64_t)K * 2};
+    cuuint64_t strides[1] = {(cuuint64_t)row_stride * 2};
     cuuint32_t box[2] = {(cuuint32_t)BK, (cuuint32_t)box_rows};
     cuuint32_t elem[2] = {1, 1};
     return fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, elem,
               CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
               CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}
+inline bool make_map(CUtensorMap* map, const void* base, long rows, int K, int box_rows) {
+    return make_map_strided(map, base, rows, K, K, box_rows);
 }
 
 }  // namespace tc5

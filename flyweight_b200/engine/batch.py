@@ -168,6 +168,28 @@ class StepBatch:
             cached = self._tiles[(tokens_per_tile, first_segment)] = (dev[:n], dev[n:], n)
         return cached
 
+    def visible_pages(self, page_size: int, first_segment: int = 0):
+        """The pages that the segments from ``first_segment`` on may see, listed one after the other: (page_seg,
+        page_no, table, n_pages), int32 on the device -- segment and logical page of every entry, and a block table
+        [S][W] that names a segment's entries by their place in the list.  Made once per step."""
+        key = ("pages", page_size, first_segment)
+        cached = self._tiles.get(key)
+        if cached is None:
+            counts = [-(-(seg.pos0 + len(seg.tokens)) // page_size) if index >= first_segment else 0
+                      for index, seg in enumerate(self.segments)]
+            n, width = sum(counts), max(counts, default=0)
+            table = np.zeros((self.n_segments, max(width, 1)), dtype=np.int32)
+            place = 0
+            for index, count in enumerate(counts):
+                table[index, :count] = np.arange(place, place + count, dtype=np.int32)
+                place += count
+            host = np.concatenate([np.repeat(np.arange(self.n_segments, dtype=np.int32), counts)]
+                                  + [np.arange(count, dtype=np.int32) for count in counts] + [table.reshape(-1)])
+            self.h2d_bytes += host.size * 4
+            dev = _to_device(host, self._device, self._pinned)
+            cached = self._tiles[key] = (dev[:n], dev[n:2 * n], dev[2 * n:].view(table.shape), n)
+        return cached
+
 
 @dataclass
 class StepContext:

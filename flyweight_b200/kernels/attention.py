@@ -41,6 +41,10 @@ def set_tcgen05_enabled(flag: bool) -> None:
 
 
 
+def tcgen05_enabled() -> bool:
+    return _use_tcgen05 and not _force_tiled
+
+
 _split_mixed = True
 
 

@@ -186,3 +186,98 @@ def latent_attention(qa: torch.Tensor, pool: torch.Tensor, sink: Optional[torch.
              ptr(batch.tok_seg), ptr(block_table), block_table.shape[1], pool.shape[2], ptr(out), T, heads,
              rank, used, row, c_float(scale), stream())
     return out
+
+
+# ------------------------------------------------------------------ rows longer than a head of the paged kernels
+SM_COUNT = 148
+ROWS_PER_CTA = 32            # query rows (heads of a token, or of neighbouring tokens) that share a tile of cached rows
+EXPAND_FROM = 64             # the longest portion of a step from which its prompts read expanded head keys and values
+EXPAND_BYTES = 2 << 30       # the most scratch those may take
+
+
+def rows_accept(rank: int, row: int, page_size: int) -> bool:
+    """Whether ``rows_attention`` has a form for such cache rows."""
+    return (page_size == 64 and row % 16 == 0 and 16 <= row <= 576 and 0 < rank <= 512 and rank <= row
+            and (row > 320 or rank <= 320) and (row > 192 or rank <= 192))
+
+
+def rows_splits(items: int, max_tiles: int, row: int):
+    """(slices of the context, 64-key tiles a slice) of a step of ``items`` = tokens x head groups: as many slices as
+    are resident at once, at least four tiles a slice.  Static sizes only, so a captured graph stays valid."""
+    resident = SM_COUNT * (2 if row <= 192 else 1)
+    splits = max(1, min(resident // max(1, items), -(-max_tiles // 4), 64))
+    splits = max(splits, -(-max_tiles // 128))
+    tiles = -(-max_tiles // splits)
+    return -(-max_tiles // tiles), tiles
+
+
+def rows_attention(qa: torch.Tensor, pool: torch.Tensor, sink: Optional[torch.Tensor], batch, block_table: torch.Tensor,
+                   rank: int, scale: float, singles: int) -> torch.Tensor:
+    """``latent_attention`` in bfloat16 on tensor cores: scores over the whole row (what lies behind the key part is
+    zero in queries and cache).  The first ``singles`` tokens are requests that decode (their context is cut into
+    slices), the segments behind them portions of prompts.  Returns [tokens of qa][heads * rank]."""
+    check_tensor("latent queries", qa, torch.bfloat16)
+    check_tensor("latent pool", pool, torch.bfloat16)
+    T, heads, row = qa.shape
+    if sink is not None:
+        check_tensor("sink", sink, torch.float32, (heads,))
+    _i32("block table", block_table)
+    out = torch.empty((T, heads * rank), dtype=qa.dtype, device=qa.device)
+    groups = -(-heads // ROWS_PER_CTA)
+    per_cta = -(-heads // groups)
+    width = block_table.shape[1]
+
+    def launch(items, tiles, tokens, splits, tiles_per_split, part_o, part_ml):
+        lib.call("fwb_latent_attention_mma", ptr(qa), ptr(pool), ptr(sink), ptr(batch.positions), ptr(batch.tok_seg),
+                 ptr(batch.seg_start), ptr(tiles[0]) if tiles else None, ptr(tiles[1]) if tiles else None,
+                 ptr(block_table), width, pool.shape[2], ptr(out), ptr(part_o), ptr(part_ml), items, heads, per_cta,
+                 tokens, rank, row, splits, tiles_per_split, c_float(scale), stream(), launches=2 if splits > 1 else 1)
+
+    if singles > 0:
+        splits, tiles_per_split = rows_splits(singles * groups, width, row)
+        part_o = part_ml = None
+        if splits > 1:
+            part_o = torch.empty((singles, heads, splits, rank), dtype=torch.float32, device=qa.device)
+            part_ml = torch.empty((singles, heads, splits, 2), dtype=torch.float32, device=qa.device)
+        launch(singles, None, 1, splits, tiles_per_split, part_o, part_ml)
+    if singles < T:
+        tokens = max(1, ROWS_PER_CTA // per_cta)
+        tile_seg, tile_tok0, n_tiles = batch.attention_tiles(tokens, singles)
+        launch(n_tiles, (tile_seg, tile_tok0), tokens, 1, width, None, None)
+    return out
+
+
+def expanded_head(dim: int, rot: int, vdim: int) -> int:
+    """The head size of the prompt kernel that takes expanded keys and values of these sizes (0: none)."""
+    used = max(dim + rot, vdim)
+    return 0 if used > 128 or (dim | rot) & 1 else (64 if used <= 64 else 128)
+
+
+def expanded_prefill(q: torch.Tensor, pool: torch.Tensor, w_kv: torch.Tensor, table: torch.Tensor, batch,
+                     block_table: torch.Tensor, heads: int, dim: int, rot: int, rot_dims: int, pairing: str, hd: int,
+                     scale: float, sink: Optional[torch.Tensor], first: int) -> torch.Tensor:
+    """The prompts of a step (the segments from ``first`` on) against head keys and values: the cached rows they may
+    see are gathered and go through one product with ``w_kv`` [2 heads hd][row] (U_h and the identity on the turned
+    part, then V_h; zero rows behind a head's own), and the tcgen05 prompt kernel reads the result in place.  q:
+    [T][heads (dim + rot)], the turned part not yet turned.  Returns [T][heads hd]; other segments' rows are undefined."""
+    from . import ops
+    check_tensor("queries", q, torch.bfloat16)
+    check_tensor("latent pool", pool, torch.bfloat16)
+    row = pool.shape[3]
+    check_tensor("expansion", w_kv, torch.bfloat16, (2 * heads * hd, row))
+    T = q.shape[0]
+    page_seg, page_no, pages, n_pages = batch.visible_pages(64, first)
+    rows = torch.empty((n_pages * 64, row), dtype=pool.dtype, device=pool.device)
+    lib.call("fwb_latent_gather", ptr(pool), ptr(page_seg), ptr(page_no), ptr(block_table), block_table.shape[1],
+             ptr(batch.seg_start), ptr(batch.seg_pos0), ptr(rows), n_pages, row, stream())
+    kv = ops.linear(rows, w_kv, torch.bfloat16)
+    spread = torch.empty((T, heads * hd), dtype=q.dtype, device=q.device)
+    lib.call("fwb_latent_spread", ptr(q), ptr(table), ptr(batch.positions), ptr(spread), T, heads, dim, rot, rot_dims,
+             ROPE_PAIRINGS[pairing], hd, stream())
+    out = torch.empty_like(spread)
+    tile_seg, tile_tok0, n_tiles = batch.attention_tiles(128, first)
+    lib.call("fwb_attention_prefill_tcgen05_rows", ptr(spread), ptr(kv), kv.data_ptr() + heads * hd * 2,
+             c_longlong(kv.shape[1]), kv.shape[0], ptr(batch.positions), ptr(batch.seg_start), ptr(tile_seg),
+             ptr(tile_tok0), ptr(pages), pages.shape[1], ptr(out), n_tiles, heads, hd, 128, c_float(scale), ptr(sink),
+             stream())
+    return out

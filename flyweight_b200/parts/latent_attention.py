@@ -18,7 +18,10 @@ In bfloat16 that attention is the engine's paged attention with one pool head th
 reads and that serves as key and as value (tcgen05 for prompt portions, the split-context kernel for
 single tokens), so the cached row is padded to a head size those kernels have (64 or 128 entries when
 it fits, which gives prompts the tcgen05 kernel); the per-head products run on tensor cores too.
-Rows longer than 128 entries, and the 32-bit path, run the fp32 kernel of ``csrc/latent_attention.cu``.
+Longer rows (up to 576 entries) have kernels of their own (``csrc/latent_rows.cu``): single tokens and short portions
+run the same absorbed form on the long rows; portions of 64 tokens and more expand the rows they may see into head
+keys and values with one product and run the tcgen05 prompt kernel on those, which costs less per pair.  The
+32-bit path runs the fp32 kernel of ``csrc/latent_attention.cu``.
 """
 from __future__ import annotations
 
@@ -26,7 +29,7 @@ import torch
 
 from ..kernels import attention as attention_kernels
 from ..kernels import latent as latent_kernels
-from ..kernels import ops
+from ..kernels import mixing, ops
 from ..weights.loader import TensorDecl
 from .base import Mixer, PagedKV, Precision, build_position, register_mixer
 
@@ -77,7 +80,9 @@ class LatentAttention(Mixer):
         self.row = 64 if used <= 64 else (128 if 96 < used <= 128 else _round_up(used, 16))
         self.q_width = self.n_heads * (self.dim + self.rot)
         self.w_in = self.w_uk_t = self.w_uv = self.w_o = self.norm_w = self.sink = self.w_gate = None
-        self.w_uq = self.q_norm_w = None
+        self.w_uq = self.q_norm_w = self.w_kv = None
+        # the head size of the prompt kernel that reads expanded keys and values of this layer (0: none)
+        self.expanded = latent_kernels.expanded_head(self.dim, self.rot, self.vdim)
 
     def declare(self):
         n, H = self.names, self.hidden
@@ -116,6 +121,8 @@ class LatentAttention(Mixer):
         self.w_uk_t = precision.matrix(uk.contiguous(), device)
         self.w_uv = precision.matrix(get(n["uv"]).reshape(self.n_heads, self.vdim, self.rank), device)
         self.w_o = precision.matrix(get(n["o"]), device)
+        if self.q_rank and self.expanded and self.row > 128 and precision.name == "bfloat16":
+            self.w_kv = self._expansion(get(n["uk"]), get(n["uv"]), device)
         if self.q_rank:
             self.w_uq = precision.matrix(get(n["uq"]), device)
             self.q_norm_w = precision.vector(get(n["dq_norm"]), device)
@@ -123,6 +130,18 @@ class LatentAttention(Mixer):
             self.norm_w = precision.vector(get(n["dkv_norm"]), device)
         if self.has_sink:
             self.sink = precision.vector(get(n["sink"]), device)
+
+    def _expansion(self, uk, uv, device):
+        """[2][heads][hd][row]: what makes head keys (U_h on the latent, the turned part as it is) and head values out of
+        a cached row; zero rows fill a head up to the prompt kernel's size.  None for matrices not in bfloat16."""
+        if uk.dtype != torch.bfloat16 or uv.dtype != torch.bfloat16:
+            return None
+        H, hd, rank = self.n_heads, self.expanded, self.rank
+        both = torch.zeros((2, H, hd, self.row), dtype=torch.bfloat16)
+        both[0, :, :self.dim, :rank] = uk.reshape(H, self.dim, rank).cpu()
+        both[0, :, self.dim:self.dim + self.rot, rank:rank + self.rot] = torch.eye(self.rot, dtype=torch.bfloat16)
+        both[1, :, :self.vdim, :rank] = uv.reshape(H, self.vdim, rank).cpu()
+        return both.view(2 * H * hd, self.row).to(device)
 
     def _matrices(self):
         return tuple(m for m in (self.w_in, self.w_uq, self.w_uk_t, self.w_uv, self.w_o, self.w_gate) if m is not None)
@@ -188,13 +207,48 @@ class LatentAttention(Mixer):
             proj, pool = ops.linear(cq, self.w_uq, act), None    # the cache row is written
         else:
             proj = ops.linear(h, self.w_in, act)                 # [T][queries | latent + key part]
+        heads_out = torch.empty((proj.shape[0], self.n_heads * self.vdim), dtype=act, device=proj.device)
+        absorbed = heads_out.shape[0]                            # the step's first tokens that read the rows as they are
+        if self._expands(ctx, cache.k_pool, proj):
+            absorbed = batch.leading_singles
+            rows = latent_kernels.expanded_prefill(
+                proj, cache.k_pool, self.w_kv, table, batch, block_table, self.n_heads, self.dim, self.rot, rot_dims,
+                pairing, self.expanded, self.scale, self.sink, absorbed)
+            if self.expanded == self.vdim:
+                heads_out = rows
+            else:
+                mixing.place_heads_(rows, self.n_heads, self.expanded, self.vdim, heads_out, 0, heads_out.shape[1])
+        if absorbed:
+            self._absorbed(ctx, proj[:absorbed], table, rot_dims, pairing, pool, cache, block_table, heads_out[:absorbed])
+        if self.gate:
+            mixing.sigmoid_gate_cols_mul_(heads_out, proj, self._gate_col, self.n_heads, self.vdim)
+        return ops.linear(heads_out, self.w_o, torch.float32)
+
+    def _expands(self, ctx, pool, proj) -> bool:
+        """Whether this step's prompts read head keys and values that one product expands from the cached rows: rows
+        too long for the paged kernels, and portions long enough to pay for it."""
+        batch = ctx.batch
+        return bool(self.w_kv is not None and batch.max_segment >= latent_kernels.EXPAND_FROM
+                    and self._long_rows(ctx, pool) and attention_kernels.tcgen05_enabled()
+                    and sum(seg.pos0 + len(seg.tokens) + 64 for seg in batch.segments) * self.w_kv.shape[0] * 2
+                    <= latent_kernels.EXPAND_BYTES)
+
+    def _long_rows(self, ctx, pool) -> bool:
+        """bfloat16 rows on tensor cores that are longer than a head of the paged kernels."""
+        return (ctx.precision.act_dtype == torch.bfloat16 and pool.dtype == torch.bfloat16
+                and latent_kernels.tensor_cores()
+                and not attention_kernels.tensor_core_shape_ok(self.n_heads, 1, self.row, pool.shape[2])
+                and latent_kernels.rows_accept(self.rank, self.row, pool.shape[2]))
+
+    def _absorbed(self, ctx, proj, table, rot_dims, pairing, pool_to_write, cache, block_table, heads_out):
+        """Every query head as a row of the cache row's layout, for the step's first tokens (the rows of ``proj``)."""
+        act, batch, pool = ctx.precision.act_dtype, ctx.batch, cache.k_pool
         qa = latent_kernels.latent_prepare(
-            proj, self.q_width, self.norm_w, table, batch, block_table,
-            pool, self.n_heads, self.dim, self.rot, rot_dims, pairing,
-            self.rank, self.row, self.eps)
+            proj, self.q_width, self.norm_w, table, batch, block_table, pool_to_write, self.n_heads, self.dim, self.rot,
+            rot_dims, pairing, self.rank, self.row, self.eps)
         qa2 = qa.view(qa.shape[0], self.n_heads * self.row)
         latent_kernels.head_linear(proj, 0, self.dim + self.rot, self.dim, self.w_uk_t, qa2, 0, self.row)
-        pool = cache.k_pool
+        stride = self.rank
         if (act == torch.bfloat16 and pool.dtype == torch.bfloat16 and latent_kernels.tensor_cores()
                 and attention_kernels.tensor_core_shape_ok(self.n_heads, 1, self.row, pool.shape[2])):
             # many query heads over one pool head whose rows are keys and values: the paged attention
@@ -202,13 +256,10 @@ class LatentAttention(Mixer):
             mixed = attention_kernels.paged_attention(ctx, qa2, cache, block_table, self.n_heads, 0, self.scale,
                                                       act, sink=self.sink)
             stride = self.row
+        elif self._long_rows(ctx, pool):
+            singles = qa.shape[0] if batch.max_segment == 1 else min(batch.leading_singles, qa.shape[0])
+            mixed = latent_kernels.rows_attention(qa, pool, self.sink, batch, block_table, self.rank, self.scale, singles)
         else:
             mixed = latent_kernels.latent_attention(qa, pool, self.sink, batch, block_table, self.rank,
                                                     self.rank + self.rot, self.scale)
-            stride = self.rank
-        heads_out = torch.empty((mixed.shape[0], self.n_heads * self.vdim), dtype=act, device=mixed.device)
         latent_kernels.head_linear(mixed, 0, stride, self.rank, self.w_uv, heads_out, 0, self.vdim)
-        if self.gate:
-            from ..kernels import mixing
-            mixing.sigmoid_gate_cols_mul_(heads_out, proj, self._gate_col, self.n_heads, self.vdim)
-        return ops.linear(heads_out, self.w_o, torch.float32)

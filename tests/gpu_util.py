@@ -11,6 +11,7 @@ import torch
 
 import plain_diforax
 import plain_fobatar
+import plain_futezen
 import plain_gukosun
 import plain_kemitar
 import plain_lfm2
@@ -23,7 +24,7 @@ P = plain_lfm2
 def plain_module(name: str):
     """The plain implementation of the tiny configuration's architecture."""
     return {"Kemitar": plain_kemitar, "Diforax": plain_diforax, "Gukosun": plain_gukosun,
-            "Fobatar": plain_fobatar, "Vugipel": plain_vugipel}.get(TINY[name].get("architecture"), plain_lfm2)
+            "Fobatar": plain_fobatar, "Futezen": plain_futezen, "Vugipel": plain_vugipel}.get(TINY[name].get("architecture"), plain_lfm2)
 
 DTYPES = ("float32", "bfloat16")
 STORED = {"float32": torch.float32, "bfloat16": torch.bfloat16}
@@ -60,6 +61,8 @@ def _edit_for(name: str, dtype: str):
     far apart (the choice then follows the corrections; the weights still follow the scores).  The
     32-bit folders keep their random corrections, so that there the scores decide.  Vugipel's router has no
     corrections: see ``_class_routers``."""
+    if TINY[name].get("architecture") == "Futezen":
+        return lambda tensors: futezen_edit(tensors, TINY[name], dtype)
     if dtype == "bfloat16" and TINY[name].get("architecture") == "Vugipel":
         return lambda tensors: _class_routers(tensors, TINY[name])
     if dtype != "bfloat16" or TINY[name].get("architecture") != "Diforax":
@@ -74,14 +77,32 @@ def _edit_for(name: str, dtype: str):
     return spread
 
 
-def _class_routers(tensors, config) -> None:
+def futezen_edit(tensors, config, dtype: str) -> None:
+    """Decay rates of a recurrence's heads from one that forgets within a token to one that remembers hundreds (a
+    stale or lost state then shows), and in 16-bit folders routers of ``_class_routers``; a norm behind a sublayer
+    must not turn what it passes there, so its weights become one number per norm (not 0: the stored weight is not
+    the factor)."""
+    for index, layer in enumerate(config["layers"]):
+        if layer["type"] == "mamba2":
+            name = f"l{index}.mix.A_log"
+            heads = tensors[name].numel()
+            tensors[name] = torch.linspace(-6.0, 1.0, heads).to(tensors[name].dtype)
+    if dtype == "bfloat16":
+        for key in tensors:
+            if key.endswith(("norm1b", "norm2b")):
+                tensors[key] = torch.full_like(tensors[key], 0.25 if key.endswith("1b") else -0.25)
+        _class_routers(tensors, config, 3.0)
+
+
+def _class_routers(tensors, config, gap: float = 1.0) -> None:
     """Routers whose scores lie far apart for every token, so that 16-bit rounding never decides a choice: each
     token's embedding carries its own ranking of a few orthogonal directions (one per expert, distinct
     coefficients), no sublayer writes into those directions, and a router's rows are the directions themselves
     (the norm's channel weights divided out)."""
     stored = tensors["embed"].dtype
     width, vocab = int(config["width"]), int(config["vocab"])
-    moe = {i: layer["mlp"]["router"]["experts"] for i, layer in enumerate(config["layers"]) if layer.get("mlp")}
+    moe = {i: layer["mlp"]["router"]["experts"] for i, layer in enumerate(config["layers"])
+           if layer.get("mlp") and layer["mlp"]["kind"] == "moe"}
     n = max(moe.values(), default=0)
     if not n:
         return
@@ -89,7 +110,7 @@ def _class_routers(tensors, config) -> None:
     basis = torch.linalg.qr(torch.randn(width, n, generator=gen, dtype=torch.float64)).Q            # [W][n]
     without = torch.eye(width, dtype=torch.float64) - basis @ basis.T
     order = torch.rand(vocab, n, generator=gen).argsort(dim=1).to(torch.float64) - (n - 1) / 2.0
-    tensors["embed"] = (tensors["embed"].to(torch.float64) @ without + order @ basis.T).to(stored)
+    tensors["embed"] = (tensors["embed"].to(torch.float64) @ without + gap * order @ basis.T).to(stored)
     for key in tensors:
         if key.endswith((".mix.o", ".left.o", ".right.o", ".down", ".o.b")):
             tensors[key] = (without @ tensors[key].to(torch.float64)).to(stored)

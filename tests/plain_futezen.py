@@ -28,6 +28,16 @@ def bf16(value):
     return value.to(torch.bfloat16).to(value.dtype)
 
 
+def dither(seed):
+    """A stand-in for ``bf16`` that loses as much, but at random: a relative error of up to half a unit in the last
+    of bfloat16's places.  Several of them show how far apart two correct 16-bit computations may lie."""
+    gen = torch.Generator().manual_seed(seed)
+
+    def lose(value):
+        return value * (1.0 + (torch.rand(value.shape, generator=gen, dtype=value.dtype) - 0.5) * 2.0 ** -8)
+    return lose
+
+
 def load_model_dir(path):
     """(config dict, name -> tensor in float64) of a model folder: the file is a little-endian header length,
     a JSON header (dtype, shape, byte range per name) and the data."""
@@ -170,7 +180,7 @@ def mamba2_mixer(h, w, prefix, m, eps, positions, rnd=same):
     T = h.shape[0]
     p = rnd(h) @ w[prefix + "in"].T
     z, u, dt = p[:, :inner], p[:, inner:2 * inner + 2 * G * n], p[:, 2 * inner + 2 * G * n:]
-    u = silu(causal_taps(u, w[prefix + "conv"], w[prefix + "conv.b"]))
+    u = rnd(silu(causal_taps(u, w[prefix + "conv"], w[prefix + "conv.b"])))
     x, b, c = u[:, :inner], u[:, inner:inner + G * n], u[:, inner + G * n:]
     dt = softplus(dt + w[prefix + "dt_bias"])
     y, _ = scalar_decay_scan(x.view(T, H, e), b.view(T, G, n), c.view(T, G, n), dt,

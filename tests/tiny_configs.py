@@ -473,5 +473,87 @@ VUGIPEL_E = {
 TINY.update({"VA": VUGIPEL_A, "VB": VUGIPEL_B, "VC": VUGIPEL_C, "VD": VUGIPEL_D, "VE": VUGIPEL_E})
 
 
+def _low_rank_latent(heads, dim, rot_dim, vdim, q_rank, kv_rank, scale, base):
+    return {"type": "latent_attention", "mixer": {
+        "heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "q_rank": q_rank, "kv_rank": kv_rank,
+        "scale": scale, "rot": {"base": base, "dims": rot_dim}}}
+
+
+def _state_space(heads, vdim, state, groups, conv, norm_groups):
+    return {"type": "mamba2", "mixer": {"heads": heads, "vdim": vdim, "state": state, "groups": groups, "conv": conv,
+                                        "norm_groups": norm_groups}}
+
+
+def _halves_attention(heads, kv_heads, dim, vdim, scale, base, dims):
+    return {"type": "attention", "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale,
+                                           "rot": {"base": base, "dims": dims}}}
+
+
+def _relu_dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def _chosen_experts(ff, experts, top, shared=None):
+    mlp = {"kind": "moe", "expert": {"ff": ff}, "router": {"experts": experts, "top": top}}
+    if shared is not None:
+        mlp["shared"] = {"ff": shared}
+    return mlp
+
+
+# Tiny Futezen configurations that differ in every size and option: keys wider and narrower than values, sizes that
+# are no multiple of 16 or 8, rotation of all and of a part of a head, cache rows from 20 entries to 304 (every
+# attention kernel), low query ranks larger and smaller than the latent's, one to three groups of state inputs, one to
+# six norm groups, states smaller and larger than a warp's share and than a run of tokens, 1 to 5 taps, one to all
+# experts a token, with and without the shared expert, layers without a feed-forward, models of one mixer only, loops
+# over the first layers, the middle, the last, a single layer four times, all layers once, and none.
+FUTEZEN_A = {
+    "architecture": "Futezen", "vocab": 203, "width": 80, "norm": {"eps": 1e-5},
+    "loop": {"start": 0, "stop": 2, "times": 2},
+    "layers": [
+        {**_state_space(6, 10, 12, 3, 3, 2), "mlp": _chosen_experts(24, 5, 2, shared=40)},
+        {**_low_rank_latent(3, 10, 4, 14, 20, 28, 0.4, 1000.0), "mlp": _relu_dense(56)},
+        {**_halves_attention(4, 2, 20, 12, 0.5, 10000.0, 8), "mlp": None},
+    ],
+}
+FUTEZEN_B = {
+    "architecture": "Futezen", "vocab": 150, "width": 96, "norm": {"eps": 1e-6},
+    "loop": {"start": 1, "stop": 2, "times": 4},
+    "layers": [
+        {**_halves_attention(3, 1, 16, 24, 0.3, 500.0, 16), "mlp": _chosen_experts(32, 4, 4)},
+        {**_state_space(4, 7, 33, 1, 1, 2), "mlp": _relu_dense(72)},
+        {**_low_rank_latent(2, 24, 8, 8, 50, 12, 0.25, 300.0), "mlp": _chosen_experts(16, 3, 1, shared=8)},
+    ],
+}
+# Sizes that the tensor-core kernels take.
+FUTEZEN_C = {
+    "architecture": "Futezen", "vocab": 288, "width": 128, "norm": {"eps": 1e-5},
+    "loop": {"start": 2, "stop": 4, "times": 2},
+    "layers": [
+        {**_low_rank_latent(6, 48, 16, 32, 96, 160, 0.18, 20000.0), "mlp": _relu_dense(192)},
+        {**_halves_attention(8, 2, 64, 64, 0.12, 1000000.0, 32), "mlp": _chosen_experts(64, 6, 2, shared=96)},
+        {**_state_space(4, 64, 64, 2, 4, 1), "mlp": _chosen_experts(32, 4, 3, shared=64)},
+        {**_low_rank_latent(20, 64, 32, 64, 64, 272, 0.1, 10000.0), "mlp": None},
+    ],
+}
+# One mixer only.
+FUTEZEN_D = {
+    "architecture": "Futezen", "vocab": 99, "width": 64, "norm": {"eps": 1e-6},
+    "layers": [{**_state_space(2, 40, 136, 2, 5, 1), "mlp": _chosen_experts(40, 3, 2, shared=16)},
+               {**_state_space(6, 16, 16, 1, 2, 6), "mlp": None},
+               {**_state_space(3, 72, 8, 3, 4, 3), "mlp": _relu_dense(24)}],
+}
+FUTEZEN_E = {
+    "architecture": "Futezen", "vocab": 140, "width": 72, "norm": {"eps": 1e-5},
+    "loop": {"start": 0, "stop": 3, "times": 1},
+    "layers": [
+        {**_low_rank_latent(5, 16, 16, 40, 32, 80, 0.3, 100.0), "mlp": _chosen_experts(48, 8, 3)},
+        {**_low_rank_latent(1, 32, 2, 16, 8, 100, 0.2, 5000.0), "mlp": _relu_dense(40)},
+        {**_halves_attention(2, 2, 32, 32, 0.2, 1000.0, 20), "mlp": _chosen_experts(24, 2, 1, shared=32)},
+    ],
+}
+
+TINY.update({"ZA": FUTEZEN_A, "ZB": FUTEZEN_B, "ZC": FUTEZEN_C, "ZD": FUTEZEN_D, "ZE": FUTEZEN_E})
+
+
 def vocab_of(config: dict) -> int:
     return int(config.get("vocab_size", config.get("vocab")))
