@@ -47,9 +47,8 @@ def causal_conv(rows: torch.Tensor, taps: torch.Tensor, state: Optional[torch.Te
                 norm_ranges=None, col0: int = 0, bias: Optional[torch.Tensor] = None, silu: bool = False,
                 out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """A causal convolution over time on C channels of ``rows`` ([T][>= col0 + C], fp32 or bf16) from column
-    ``col0`` on, ``taps`` fp32
-    [C][n] with the last tap on the token itself: ``y[t] = sum_j taps[:, j] * rows[t - n + 1 + j]`` along each
-    request's tokens.  ``state``: fp32 [slots][n - 1][C], every live request's last n - 1 inputs (zero when it
+    ``col0`` on, ``taps`` fp32 [C][n] with the last tap on the token itself: ``y[t] = sum_j taps[:, j] *
+    rows[t - n + 1 + j]`` along each request's tokens.  ``state``: fp32 [slots][n - 1][C], every live request's last n - 1 inputs (zero when it
     starts), read in front of a portion and moved on by this call (None when n == 1).  ``norm_ranges``: one or two
     ``(col0, weight, count, eps)`` as ``rmsnorm_ranges_`` takes them; those column ranges of the result are
     normed by the same launch.  ``bias``: fp32 [C], added to the convolved value; ``silu``: which then passes silu.
@@ -74,11 +73,11 @@ def causal_conv(rows: torch.Tensor, taps: torch.Tensor, state: Optional[torch.Te
         if not 1 <= len(norm_ranges) <= 2 or C * 4 > 160 * 1024:
             raise KernelError("the convolution norms one or two column ranges of rows of at most 40,960 channels")
         eps = float(norm_ranges[0][3])
-        for index, (col0, weight, count, this_eps) in enumerate(norm_ranges):
+        for index, (first, weight, count, this_eps) in enumerate(norm_ranges):
             check_tensor("range norm weight", weight, torch.float32)
             if float(this_eps) != eps:
                 raise KernelError("the ranges of one launch share their eps")
-            norm_args[4 * index:4 * index + 4] = [int(col0), weight.numel(), int(count), ptr(weight)]
+            norm_args[4 * index:4 * index + 4] = [int(first), weight.numel(), int(count), ptr(weight)]
     out = torch.empty((T, C), dtype=out_dtype or rows.dtype, device=rows.device)
     lib.call("fwb_causal_conv", ptr(rows), ptr(out), is_bf16(rows), is_bf16(out), ptr(bias), 1 if silu else 0,
              c_longlong(ld), c_longlong(C), int(col0), C, ptr(taps), n,

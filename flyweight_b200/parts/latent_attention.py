@@ -45,9 +45,9 @@ class LatentAttention(Mixer):
     whose ``rotary_dim`` <= rot_dim), sink (True: a learned number per head joins the softmax
     denominator), shares_cache (True: reads the rows of another execution; no latent projection), gate
     ("head": tensor ``g`` [heads][H], every head's output times sigmoid(g h) of its head, from the mixer's
-    own input), q_rank (> 0: the queries come from a
-    low-rank row that is RMS-normed with a weight in between, q = W_uq (w * unit(W_dq h)); tensors dq [q_rank][H],
-    dq_norm [q_rank], uq instead of q).  tensors: q, dkv, dkv_norm, uk, uv, o, sink, g."""
+    own input), q_rank (> 0: the queries come from a low-rank row that is RMS-normed with a weight in between,
+    q = W_uq (w * unit(W_dq h)); tensors dq [q_rank][H], dq_norm [q_rank], uq instead of q).  tensors: q, dkv,
+    dkv_norm, uk, uv, o, sink, g."""
     graph_safe = True
 
     def __init__(self, spec):
@@ -86,15 +86,14 @@ class LatentAttention(Mixer):
 
     def declare(self):
         n, H = self.names, self.hidden
-        out = {n["uk"]: TensorDecl((self.n_heads * self.dim, self.rank)),
-               n["uv"]: TensorDecl((self.n_heads * self.vdim, self.rank)),
-               n["o"]: TensorDecl((H, self.n_heads * self.vdim))}
         if self.q_rank:
-            out[n["dq"]] = TensorDecl((self.q_rank, H))
-            out[n["dq_norm"]] = TensorDecl((self.q_rank,), "norm")
-            out[n["uq"]] = TensorDecl((self.q_width, self.q_rank))
+            out = {n["dq"]: TensorDecl((self.q_rank, H)), n["dq_norm"]: TensorDecl((self.q_rank,), "norm"),
+                   n["uq"]: TensorDecl((self.q_width, self.q_rank))}
         else:
-            out[n["q"]] = TensorDecl((self.q_width, H))
+            out = {n["q"]: TensorDecl((self.q_width, H))}
+        out.update({n["uk"]: TensorDecl((self.n_heads * self.dim, self.rank)),
+                    n["uv"]: TensorDecl((self.n_heads * self.vdim, self.rank)),
+                    n["o"]: TensorDecl((H, self.n_heads * self.vdim))})
         if not self.shares_cache:
             out[n["dkv"]] = TensorDecl((self.rank + self.rot, H))
             out[n["dkv_norm"]] = TensorDecl((self.rank,), "norm")
