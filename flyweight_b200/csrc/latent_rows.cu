@@ -6,9 +6,10 @@
 //                      latent's space), against the cached rows themselves; values are a row's first `rank` columns.
 //                      mma.sync m16n8k16, fp32 accumulation and softmax.  One CTA takes 16 or 32 query rows (heads
 //                      of one token, or of a few neighbouring tokens) and one slice of the context, 64 keys at a
-//                      time: a cached row is read once for all of them.  Eight warps share a tile's scores (16 rows
-//                      by 8 or 16 keys each, the queries in registers), the scores meet in shared memory for the
-//                      online softmax, and for the weighted sum every warp owns a share of the latent's columns.
+//                      time: a cached row is read once for all of them.  Eight or sixteen warps share a tile's
+//                      scores (16 rows by 8 or 16 keys each, the queries in registers), the scores meet in shared
+//                      memory for the online softmax, and for the weighted sum every warp owns a share of the
+//                      latent's columns.
 //                      Slices are merged by a second kernel through fp32 scratch.  Steps of single tokens, and
 //                      prompts whose heads fit no prompt kernel.
 //   fwb_latent_gather  the cached rows that the prompts of a step may see, side by side and padded to runs of 64
@@ -23,8 +24,6 @@ using namespace fwb;
 namespace {
 
 constexpr int KEYS = 64;               // keys per tile == page size
-constexpr int THREADS = 256;
-constexpr int WARPS = 8;
 constexpr int PAD = 8;                 // bf16 entries behind a shared row (rows then start 4 banks apart)
 constexpr int PS = KEYS + 8;           // bf16 entries of a row of probabilities
 constexpr int SS = KEYS + 4;           // fp32 entries of a row of scores
@@ -43,10 +42,6 @@ __device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const __nv_bfloat16* row
     const uint32_t at = (uint32_t)__cvta_generic_to_shared(row);
     asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(at));
-}
-__device__ __forceinline__ void ldsm2(uint32_t (&r)[2], const __nv_bfloat16* row) {
-    const uint32_t at = (uint32_t)__cvta_generic_to_shared(row);
-    asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(at));
 }
 __device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], const __nv_bfloat16* row) {
     const uint32_t at = (uint32_t)__cvta_generic_to_shared(row);
@@ -77,12 +72,16 @@ struct RowsParams {
     float scale_log2;
 };
 
-// MT: bands of 16 query rows.  KS: the most 16-entry steps of a row.  NB: 16-column blocks of the latent a warp owns.
-template <int MT, int KS, int NB>
-__global__ void __launch_bounds__(THREADS, KS <= 12 ? 2 : 1)
+// MT: bands of 16 query rows.  KS: the most 16-entry steps of a row (steps behind a shorter row's last repeat it
+// against zero queries: no branch in the loop).  NB: 16-column blocks of the latent a warp owns.
+template <int MT, int KS, int NB, int WARPS>
+__global__ void __launch_bounds__(WARPS * 32, WARPS == 8 && KS <= 18 && MT == 1 ? 2 : 1)
 latent_rows_kernel(const RowsParams prm) {
     fwb::pdl_entry();
-    constexpr int M = MT * 16, NT = MT, OWN = M / WARPS;    // NT: 8-key tiles of a warp's scores; OWN: rows of its softmax
+    constexpr int THREADS = WARPS * 32, M = MT * 16;
+    constexpr int NT = MT * 8 / WARPS, OWN = M / WARPS;     // 8-key tiles of a warp's scores; rows of its softmax
+    constexpr int STEPS = KS * 16;
+    constexpr int LPR = 32 / OWN, PER = KEYS / LPR;         // lanes of a row's softmax, scores a lane
     extern __shared__ __align__(16) uint8_t smem_raw[];
     const int row = prm.row, RS = row + PAD, rank = prm.rank;
     __nv_bfloat16* Ks = reinterpret_cast<__nv_bfloat16*>(smem_raw);             // [stages][KEYS][RS]
@@ -120,6 +119,7 @@ latent_rows_kernel(const RowsParams prm) {
 
     // this warp's part of the scores: 16 rows by NT * 8 keys
     const int mt0 = MT == 2 ? (warp & 1) : 0, key0 = (MT == 2 ? (warp >> 1) : warp) * NT * 8;
+    static_assert(NT == 1 || NT == 2, "a warp scores 8 or 16 keys of a tile");
     uint32_t qf[KS][4];
     {
         size_t lo = 0, hi = 0;
@@ -136,18 +136,17 @@ latent_rows_kernel(const RowsParams prm) {
             qf[k][3] = in && has_hi ? *reinterpret_cast<const uint32_t*>(q_hi + d + 8) : 0u;
         }
     }
-    // this warp's rows of the softmax: running maximum, a lane's share of the running sum, last visible key
-    float m_run[OWN], l_run[OWN];
-    int hi_key[OWN];
-#pragma unroll
-    for (int i = 0; i < OWN; ++i) {
-        const int r = warp * OWN + i;
-        size_t at = 0;
-        const bool valid = row_at(r, at);
-        hi_key[i] = valid ? prm.positions[tok0 + r / nh] : -1;
-        const bool start = valid && prm.sink && split == 0;
-        m_run[i] = start ? prm.sink[h0 + r % nh] * LOG2E : -INFINITY;
-        l_run[i] = start && lane == 0 ? 1.0f : 0.0f;
+    // this lane's row of the softmax (LPR lanes share one): running maximum, a lane's share of the running sum, last
+    // visible key
+    const int own = warp * OWN + lane / LPR, sub = lane % LPR;
+    float m_run = -INFINITY, l_run = 0.0f;
+    int hi_key = -1;
+    if (own < rows) {
+        hi_key = prm.positions[tok0 + own / nh];
+        if (prm.sink && split == 0) {
+            m_run = prm.sink[h0 + own % nh] * LOG2E;
+            l_run = sub == 0 ? 1.0f : 0.0f;
+        }
     }
     float acc[MT][NB][2][4];
 #pragma unroll
@@ -157,16 +156,22 @@ latent_rows_kernel(const RowsParams prm) {
 #pragma unroll
             for (int j = 0; j < 8; ++j) acc[mt][nb][j >> 2][j & 3] = 0.0f;
 
-    const int chunks = row >> 3;
+    const int chunks = row >> 3, row_step = THREADS / chunks, chunk_step = THREADS % chunks;
+    const int row_first = threadIdx.x / chunks, chunk_first = threadIdx.x % chunks;
     auto issue = [&](int tile) {
         if (tile < last) {
             __nv_bfloat16* dst = Ks + (size_t)((tile - first) % prm.stages) * KEYS * RS;
             const __nv_bfloat16* src = prm.pool + (size_t)table[tile] * KEYS * row;
             const int seen = pos_last - tile * KEYS + 1;    // rows behind the last visible key are zero
-            for (int i = threadIdx.x; i < KEYS * chunks; i += THREADS) {
-                const int r = i / chunks, c = (i - r * chunks) << 3;
-                if (r < seen) cp_async16(dst + r * RS + c, src + (size_t)r * row + c);
-                else *reinterpret_cast<uint4*>(dst + r * RS + c) = make_uint4(0u, 0u, 0u, 0u);
+            for (int r = row_first, c = chunk_first; r < KEYS;) {
+                if (r < seen) cp_async16(dst + r * RS + c * 8, src + r * row + c * 8);
+                else *reinterpret_cast<uint4*>(dst + r * RS + c * 8) = make_uint4(0u, 0u, 0u, 0u);
+                r += row_step;
+                c += chunk_step;
+                if (c >= chunks) {
+                    c -= chunks;
+                    ++r;
+                }
             }
         }
         cp_async_commit();
@@ -182,24 +187,26 @@ latent_rows_kernel(const RowsParams prm) {
             float s[2][NT][4];
 #pragma unroll
             for (int j = 0; j < 2 * NT * 4; ++j) s[j / (NT * 4)][(j >> 2) % NT][j & 3] = 0.0f;
-            if (MT == 2) {
+            if (NT == 2) {
                 const __nv_bfloat16* kb = kt + (key0 + (lane & 7) + ((lane >> 4) << 3)) * RS + (((lane >> 3) & 1) << 3);
 #pragma unroll
                 for (int k = 0; k < KS; ++k) {
-                    if (k * 16 >= row) break;
                     uint32_t b[4];
-                    ldsm4(b, kb + k * 16);
+                    ldsm4(b, kb + (STEPS == row || k * 16 < row ? k * 16 : row - 16));
                     mma_bf16(s[k & 1][0], qf[k], b[0], b[1]);
                     mma_bf16(s[k & 1][NT - 1], qf[k], b[2], b[3]);
                 }
             } else {
-                const __nv_bfloat16* kb = kt + (key0 + (lane & 7)) * RS + (((lane >> 3) & 1) << 3);
+                // 8 keys by two steps at a time
+                const __nv_bfloat16* kb = kt + (key0 + (lane & 7)) * RS;
+                const int at = (lane >> 3) << 3;
 #pragma unroll
-                for (int k = 0; k < KS; ++k) {
-                    if (k * 16 >= row) break;
-                    uint32_t b[2];
-                    ldsm2(b, kb + k * 16);
-                    mma_bf16(s[k & 1][0], qf[k], b[0], b[1]);
+                for (int k = 0; k < KS; k += 2) {
+                    uint32_t b[4];
+                    const int c = k * 16 + at;
+                    ldsm4(b, kb + (c < row ? c : row - 8));
+                    mma_bf16(s[0][0], qf[k], b[0], b[1]);
+                    mma_bf16(s[1][0], qf[k + 1], b[2], b[3]);
                 }
             }
 #pragma unroll
@@ -210,19 +217,39 @@ latent_rows_kernel(const RowsParams prm) {
                         make_float2(s[0][nt][2 * half] + s[1][nt][2 * half], s[0][nt][2 * half + 1] + s[1][nt][2 * half + 1]);
         }
         __syncthreads();
+        {
+            // groups of four neighbouring keys, LPR groups apart
+            float v[PER];
+            float top = -INFINITY;
 #pragma unroll
-        for (int i = 0; i < OWN; ++i) {
-            const int r = warp * OWN + i, key = tile * KEYS + lane;
-            const float v0 = key <= hi_key[i] ? Sc[r * SS + lane] * prm.scale_log2 : -INFINITY;
-            const float v1 = key + 32 <= hi_key[i] ? Sc[r * SS + lane + 32] * prm.scale_log2 : -INFINITY;
-            const float m_new = fmaxf(m_run[i], warp_max(fmaxf(v0, v1)));
+            for (int j = 0; j < PER; j += 4) {
+                const int c = 4 * (sub + (j / 4) * LPR);
+                const float4 s4 = *reinterpret_cast<const float4*>(Sc + own * SS + c);
+                const int left = hi_key - (tile * KEYS + c);                // visible: key c + i with i <= left
+                v[j] = left >= 0 ? s4.x * prm.scale_log2 : -INFINITY;
+                v[j + 1] = left >= 1 ? s4.y * prm.scale_log2 : -INFINITY;
+                v[j + 2] = left >= 2 ? s4.z * prm.scale_log2 : -INFINITY;
+                v[j + 3] = left >= 3 ? s4.w * prm.scale_log2 : -INFINITY;
+                top = fmaxf(fmaxf(top, fmaxf(v[j], v[j + 1])), fmaxf(v[j + 2], v[j + 3]));
+            }
+#pragma unroll
+            for (int step = LPR / 2; step > 0; step >>= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, step));
+            const float m_new = fmaxf(m_run, top);
             const float base = m_new == -INFINITY ? 0.0f : m_new;           // a row that has seen no key yet
-            const float p0 = exp2f(v0 - base), p1 = exp2f(v1 - base), corr = exp2f(m_run[i] - base);
-            l_run[i] = fmaf(l_run[i], corr, p0 + p1);
-            m_run[i] = m_new;
-            Ps[r * PS + lane] = __float2bfloat16_rn(p0);
-            Ps[r * PS + lane + 32] = __float2bfloat16_rn(p1);
-            if (lane == 0) corr_s[r] = corr;
+            const float corr = exp2f(m_run - base);
+            float sum = 0.0f;
+#pragma unroll
+            for (int j = 0; j < PER; j += 4) {
+                const float p0 = exp2f(v[j] - base), p1 = exp2f(v[j + 1] - base);
+                const float p2 = exp2f(v[j + 2] - base), p3 = exp2f(v[j + 3] - base);
+                sum += (p0 + p1) + (p2 + p3);
+                const __nv_bfloat162 lo = __floats2bfloat162_rn(p0, p1), hi = __floats2bfloat162_rn(p2, p3);
+                *reinterpret_cast<uint2*>(Ps + own * PS + 4 * (sub + (j / 4) * LPR)) =
+                    make_uint2(*reinterpret_cast<const uint32_t*>(&lo), *reinterpret_cast<const uint32_t*>(&hi));
+            }
+            l_run = fmaf(l_run, corr, sum);
+            m_run = m_new;
+            if (sub == 0) corr_s[own] = corr;
         }
         __syncthreads();
 #pragma unroll
@@ -246,8 +273,8 @@ latent_rows_kernel(const RowsParams prm) {
                 ldsm4(p[mt], Ps + (mt * 16 + (lane & 15)) * PS + kk * 16 + ((lane >> 4) << 3));
 #pragma unroll
             for (int nb = 0; nb < NB; ++nb) {
-                const int col = (warp + WARPS * nb) * 16;
-                if (col >= rank) break;
+                // (a block behind the last column repeats that one; nobody stores its sums)
+                const int col = (warp + WARPS * nb) * 16 < row ? (warp + WARPS * nb) * 16 : row - 16;
                 uint32_t b[4];
                 ldsm4t(b, kt + (kk * 16 + (lane & 15)) * RS + col + ((lane >> 4) << 3));
 #pragma unroll
@@ -260,12 +287,10 @@ latent_rows_kernel(const RowsParams prm) {
     }
     cp_async_wait<0>();
 #pragma unroll
-    for (int i = 0; i < OWN; ++i) {
-        const float l = warp_sum(l_run[i]);
-        if (lane == 0) {
-            l_s[warp * OWN + i] = l;
-            m_s[warp * OWN + i] = m_run[i];
-        }
+    for (int step = LPR / 2; step > 0; step >>= 1) l_run += __shfl_xor_sync(0xffffffffu, l_run, step);
+    if (sub == 0) {
+        l_s[own] = l_run;
+        m_s[own] = m_run;
     }
     __syncthreads();
     const bool whole = prm.splits == 1;
@@ -381,15 +406,15 @@ size_t rows_smem(int mt, int row, int stages) {
     return (size_t)stages * KEYS * (row + PAD) * 2 + m * PS * 2 + m * SS * 4 + 3 * m * 4;
 }
 
-template <int MT, int KS, int NB>
+template <int MT, int KS, int NB, int WARPS>
 int launch_rows(RowsParams prm, int items, int groups, cudaStream_t stream) {
-    constexpr size_t LIMIT = KS <= 12 ? 112 * 1024 : 224 * 1024;
+    constexpr size_t LIMIT = WARPS == 8 && KS <= 18 && MT == 1 ? 112 * 1024 : 224 * 1024;
     prm.stages = rows_smem(MT, prm.row, 3) <= LIMIT ? 3 : 2;
     const size_t smem = rows_smem(MT, prm.row, prm.stages);
-    auto kernel = latent_rows_kernel<MT, KS, NB>;
+    auto kernel = latent_rows_kernel<MT, KS, NB, WARPS>;
     cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
-    fwb::pdl(kernel, dim3(items, groups, prm.splits), THREADS, smem, stream)(prm);
+    fwb::pdl(kernel, dim3(items, groups, prm.splits), WARPS * 32, smem, stream)(prm);
     return fwb_launch_status();
 }
 
@@ -446,9 +471,14 @@ FWB_API int fwb_latent_attention_mma(const void* qa, const void* pool, const flo
     prm.scale_log2 = scale * LOG2E;
     const bool two = heads_per_cta * prm.tokens_per_tile > 16;
     int status;
-    if (row <= 192) status = two ? launch_rows<2, 12, 2>(prm, n_items, groups, stream) : launch_rows<1, 12, 2>(prm, n_items, groups, stream);
-    else if (row <= 320) status = two ? launch_rows<2, 20, 3>(prm, n_items, groups, stream) : launch_rows<1, 20, 3>(prm, n_items, groups, stream);
-    else status = two ? launch_rows<2, 36, 4>(prm, n_items, groups, stream) : launch_rows<1, 36, 4>(prm, n_items, groups, stream);
+    if (row <= 192)
+        status = two ? launch_rows<2, 12, 1, 16>(prm, n_items, groups, stream) : launch_rows<1, 12, 2, 8>(prm, n_items, groups, stream);
+    else if (row <= 288 && rank <= 256)
+        status = two ? launch_rows<2, 18, 1, 16>(prm, n_items, groups, stream) : launch_rows<1, 18, 2, 8>(prm, n_items, groups, stream);
+    else if (row <= 320)
+        status = two ? launch_rows<2, 20, 3, 8>(prm, n_items, groups, stream) : launch_rows<1, 20, 3, 8>(prm, n_items, groups, stream);
+    else
+        status = two ? launch_rows<2, 36, 4, 8>(prm, n_items, groups, stream) : launch_rows<1, 36, 4, 8>(prm, n_items, groups, stream);
     if (status != FWB_OK || splits == 1) return status;
     fwb::pdl(latent_rows_merge_kernel, dim3((unsigned)((size_t)n_items * heads)), 128, 0, stream)(
         part_o, part_ml, static_cast<__nv_bfloat16*>(out), splits, rank);

@@ -164,12 +164,17 @@ template <bool VEC>
 __device__ __forceinline__ void load_rows(__nv_bfloat16* dst, int ld, const __nv_bfloat16* __restrict__ src,
                                           long long stride, int count, int width, int padded) {
     if constexpr (VEC) {
-        const int chunks = padded >> 3;
-        for (int i = threadIdx.x; i < RUN * chunks; i += THREADS) {
-            const int tok = i / chunks, c = (i - tok * chunks) << 3;
-            __nv_bfloat16* at = dst + tok * ld + c;
-            if (tok < count && c < width) cp_async16(at, src + (size_t)tok * stride + c);
+        const int chunks = padded >> 3, tok_step = THREADS / chunks, chunk_step = THREADS % chunks;
+        for (int tok = threadIdx.x / chunks, c = threadIdx.x % chunks; tok < RUN;) {
+            __nv_bfloat16* at = dst + tok * ld + c * 8;
+            if (tok < count && c * 8 < width) cp_async16(at, src + tok * stride + c * 8);
             else *reinterpret_cast<uint4*>(at) = make_uint4(0u, 0u, 0u, 0u);
+            tok += tok_step;
+            c += chunk_step;
+            if (c >= chunks) {
+                c -= chunks;
+                ++tok;
+            }
         }
     } else {
         for (int i = threadIdx.x; i < RUN * padded; i += THREADS) {
@@ -222,6 +227,16 @@ state_runs_kernel(const __nv_bfloat16* __restrict__ u, long long u_stride, const
     const float* front = SUMS ? nullptr : (head && tail ? mine : held);
     float* behind = SUMS ? held : (tail ? mine : nullptr);
     float total = 0.0f;                                // logarithm of the piece's decay so far (warp 0)
+    // warp 0 turns a run's step inputs into decays; it asks for them one run ahead
+    float ahead[2];
+    auto ask = [&](int t0) {
+#pragma unroll
+        for (int k = 0; k < 2; ++k) {
+            const int tok = t0 + lane + 32 * k;
+            ahead[k] = tok < last ? raw[(size_t)tok * raw_stride + h] : 0.0f;
+        }
+    };
+    if (warp == 0) ask(first);
 
     float S[MT][CT / 8][4];                            // rows (mt*8 + warp)*16 + g (+8), columns nt*8 + 2t (+1)
 #pragma unroll
@@ -247,9 +262,10 @@ state_runs_kernel(const __nv_bfloat16* __restrict__ u, long long u_stride, const
 #pragma unroll
             for (int k = 0; k < 2; ++k) {
                 const int tok = lane + 32 * k;
-                dt[k] = tok < m ? softplus_f32(raw[(size_t)(t0 + tok) * raw_stride + h] + bias) : 0.0f;
+                dt[k] = tok < m ? softplus_f32(ahead[k] + bias) : 0.0f;
                 sum[k] = -a * dt[k];
             }
+            ask(t0 + RUN);
 #pragma unroll
             for (int step = 1; step < 32; step <<= 1)
 #pragma unroll

@@ -201,10 +201,11 @@ def rows_accept(rank: int, row: int, page_size: int) -> bool:
             and (row > 320 or rank <= 320) and (row > 192 or rank <= 192))
 
 
-def rows_splits(items: int, max_tiles: int, row: int):
-    """(slices of the context, 64-key tiles a slice) of a step of ``items`` = tokens x head groups: as many slices as
-    are resident at once, at least four tiles a slice.  Static sizes only, so a captured graph stays valid."""
-    resident = SM_COUNT * (2 if row <= 192 else 1)
+def rows_splits(items: int, max_tiles: int, row: int, per_cta: int = ROWS_PER_CTA):
+    """(slices of the context, 64-key tiles a slice) of a step of ``items`` = tokens x head groups of ``per_cta`` heads:
+    as many slices as are resident at once, at least four tiles a slice.  Static sizes only, so a captured graph
+    stays valid."""
+    resident = SM_COUNT * (2 if per_cta <= 16 and row <= 288 else 1)
     splits = max(1, min(resident // max(1, items), -(-max_tiles // 4), 64))
     splits = max(splits, -(-max_tiles // 128))
     tiles = -(-max_tiles // splits)
@@ -234,7 +235,7 @@ def rows_attention(qa: torch.Tensor, pool: torch.Tensor, sink: Optional[torch.Te
                  tokens, rank, row, splits, tiles_per_split, c_float(scale), stream(), launches=2 if splits > 1 else 1)
 
     if singles > 0:
-        splits, tiles_per_split = rows_splits(singles * groups, width, row)
+        splits, tiles_per_split = rows_splits(singles * groups, width, row, per_cta)
         part_o = part_ml = None
         if splits > 1:
             part_o = torch.empty((singles, heads, splits, rank), dtype=torch.float32, device=qa.device)

@@ -9,6 +9,9 @@
     python -m flyweight_b200.kernels.microbench causal-conv --tokens 16384
     python -m flyweight_b200.kernels.microbench gated-average --tokens 2048
     python -m flyweight_b200.kernels.microbench route --tokens 2048
+    python -m flyweight_b200.kernels.microbench state-space --tokens 2048
+    python -m flyweight_b200.kernels.microbench latent-decode --batch 64 --context 4096
+    python -m flyweight_b200.kernels.microbench latent-prefill --tokens 2048
     python -m flyweight_b200.kernels.microbench sample --rows 8 --top-k 40
 
 It is what the ncu summaries under ``profiles/`` were captured from (small cases of the same
@@ -284,6 +287,94 @@ def run_gated_average(args) -> dict:
             "gb_s": moved / us / 1e3}
 
 
+def run_state_space(args) -> dict:
+    """The state-space recurrence over ``batch`` segments of ``tokens`` tokens (1: a decode step)."""
+    from ..engine.batch import Segment, StepBatch
+    from . import state_space
+    H, G, n, e, T = args.heads, args.groups, args.state, args.vdim, args.batch * args.tokens
+    dev = torch.device("cuda", 0)
+    width = H * e + 2 * G * n
+    state_bytes = args.batch * H * n * e * 4
+    row_bytes = T * (width * 2 + H * 4 + H * e * 4)
+    copies = max(1, min(16, -(-(256 << 20) // (row_bytes + state_bytes))))
+    us_, ps, states = ([torch.randn(shape, device=dev).to(dtype) for _ in range(copies)]
+                       for shape, dtype in (((T, width), torch.bfloat16), ((T, H), torch.float32),
+                                            ((args.batch, H * n * e), torch.float32)))
+    small = torch.zeros(H, device=dev)
+    batch = StepBatch([Segment(f"r{i}", i, 0, [0] * args.tokens, []) for i in range(args.batch)],
+                      [[[0]] * args.batch], dev)
+
+    def steps():
+        for u, p, state in zip(us_, ps, states):
+            state_space.state_space(u, p, 0, small, small, small, state, batch, H, G, n, e,
+                                    runs=False if args.scan else None)
+
+    us = _time_graph(steps, args.repeat) / copies
+    # the recurrence itself: two passes over the state a token (decay and write, read-out)
+    return {"kernel": "state_space", "batch": args.batch, "tokens": args.tokens, "heads": H, "groups": G, "state": n,
+            "vdim": e, "us": us, "gb_s": (row_bytes + 2 * state_bytes) / us / 1e3, "tflops": 4.0 * T * H * n * e / us / 1e6}
+
+
+def _latent_case(args, contexts, tokens):
+    """Pools (rotated through enough copies to exceed L2), a batch and its block table for latent rows."""
+    from ..engine.batch import Segment, StepBatch
+    dev = torch.device("cuda", 0)
+    row = -(-(args.rank + args.rot) // 16) * 16
+    pages = [-(-c // 64) for c in contexts]
+    pool_bytes = sum(pages) * 64 * row * 2
+    copies = max(1, min(16, -(-(256 << 20) // pool_bytes)))
+    pools = [torch.randn((sum(pages), 1, 64, row), device=dev).to(torch.bfloat16) for _ in range(copies)]
+    table, at = [], 0
+    for n in pages:
+        table.append(list(range(at, at + n)) + [-1] * (max(pages) - n))
+        at += n
+    batch = StepBatch([Segment(f"r{i}", i, c - tokens, [0] * tokens, []) for i, c in enumerate(contexts)], [table], dev)
+    return row, pools, batch
+
+
+def run_latent_decode(args) -> dict:
+    """Single tokens of ``batch`` requests over ``context`` cached latent rows each."""
+    from . import latent
+    row, pools, batch = _latent_case(args, [args.context] * args.batch, 1)
+    qa = torch.randn((args.batch, args.heads, row), device="cuda").to(torch.bfloat16)
+
+    def steps():
+        for pool in pools:
+            latent.rows_attention(qa, pool, None, batch, batch.block_tables[0], args.rank, 0.1, args.batch)
+
+    us = _time_graph(steps, args.repeat) / len(pools)
+    moved = args.batch * args.context * row * 2
+    return {"kernel": "latent_rows", "batch": args.batch, "context": args.context, "heads": args.heads, "row": row,
+            "us": us, "gb_s": moved / us / 1e3,
+            "tflops": 2.0 * args.batch * args.context * args.heads * (row + args.rank) / us / 1e6}
+
+
+def run_latent_prefill(args) -> dict:
+    """One prompt of ``tokens`` tokens over its own latent rows: expanded head keys and values, or the rows."""
+    from . import latent
+    row, pools, batch = _latent_case(args, [args.tokens], args.tokens)
+    heads, dim, rot, vdim = args.heads, args.dim, args.rot, args.vdim
+    hd = latent.expanded_head(dim, rot, vdim)
+    w_kv = torch.randn((2 * heads * hd, row), device="cuda").to(torch.bfloat16)
+    q = torch.randn((args.tokens, heads * (dim + rot)), device="cuda").to(torch.bfloat16)
+    qa = torch.randn((args.tokens, heads, row), device="cuda").to(torch.bfloat16)
+    table = torch.randn((args.tokens, rot // 2, 2), device="cuda")
+
+    def steps():
+        for pool in pools:
+            if args.rows:
+                latent.rows_attention(qa, pool, None, batch, batch.block_tables[0], args.rank, 0.1, 0)
+            else:
+                latent.expanded_prefill(q, pool, w_kv, table, batch, batch.block_tables[0], heads, dim, rot, rot,
+                                        "interleaved", hd, 0.1, None, 0)
+
+    steps()
+    us = _time_graph(steps, args.repeat) / len(pools)
+    per_pair = row + args.rank if args.rows else dim + rot + vdim
+    return {"kernel": "latent_rows prompt" if args.rows else "latent expanded prompt", "tokens": args.tokens,
+            "heads": heads, "us": us, "tflops": 1.0 * args.tokens ** 2 * heads * per_pair / us / 1e6}
+
+
 def run_route(args) -> dict:
     """The router of routed experts: scores of ``outputs`` outputs and the choice of ``top``."""
     from . import experts
@@ -443,6 +534,25 @@ def main(argv=None) -> int:
     rt.add_argument("--top", type=int, default=8)
     rt.add_argument("--simt", action="store_true", help="the fp32-FMA kernel at every size")
     rt.add_argument("--scores", default="sigmoid")
+    ssm = sub.add_parser("state-space")
+    ssm.add_argument("--batch", type=int, default=1)
+    ssm.add_argument("--tokens", type=int, default=2048)
+    ssm.add_argument("--heads", type=int, default=64)
+    ssm.add_argument("--groups", type=int, default=1)
+    ssm.add_argument("--state", type=int, default=128)
+    ssm.add_argument("--vdim", type=int, default=64)
+    ssm.add_argument("--scan", action="store_true", help="the token-by-token kernel")
+    for name in ("latent-decode", "latent-prefill"):
+        lat = sub.add_parser(name)
+        lat.add_argument("--batch", type=int, default=64)
+        lat.add_argument("--context", type=int, default=4096)
+        lat.add_argument("--tokens", type=int, default=2048)
+        lat.add_argument("--heads", type=int, default=32)
+        lat.add_argument("--rank", type=int, default=256)
+        lat.add_argument("--rot", type=int, default=32)
+        lat.add_argument("--dim", type=int, default=64)
+        lat.add_argument("--vdim", type=int, default=64)
+        lat.add_argument("--rows", action="store_true", help="prompt: over the rows themselves")
     smp = sub.add_parser("sample")
     smp.add_argument("--rows", type=int, default=8)
     smp.add_argument("--vocab", type=int, default=65536)
@@ -458,7 +568,8 @@ def main(argv=None) -> int:
               "attention-prefill": run_attention_prefill, "shortconv": run_shortconv,
               "causal-conv": run_causal_conv,
               "qk-norm-rope": run_qk_norm_rope, "sample": run_sample, "delta-rule": run_delta_rule,
-              "linear-attention": run_linear_attention, "gated-average": run_gated_average, "route": run_route}[args.kernel]
+              "linear-attention": run_linear_attention, "gated-average": run_gated_average, "route": run_route,
+              "state-space": run_state_space, "latent-decode": run_latent_decode, "latent-prefill": run_latent_prefill}[args.kernel]
     print(json.dumps(runner(args)))
     return 0
 

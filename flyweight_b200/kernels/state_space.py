@@ -14,11 +14,11 @@ RUNS_FROM = 16             # the longest portion of a step from which it is used
 PIECES = (128, 256, 512, 1024)
 
 
-def piece_tokens(longest: int, heads: int) -> int:
-    """Tokens of a segment that one block of the tensor-core form walks: the longest piece that still makes
-    two blocks an SM out of the step's longest segment (a shorter piece costs a pass over its tokens for its sum)."""
+def piece_tokens(tokens: int, heads: int) -> int:
+    """Tokens of a segment that one block of the tensor-core form walks: the longest piece that still makes two blocks
+    an SM out of the step's tokens (a segment of several pieces costs a second pass over its tokens, for their sums)."""
     for piece in reversed(PIECES):
-        if -(-longest // piece) * heads >= 2 * SM_COUNT:
+        if -(-tokens // piece) * heads >= 2 * SM_COUNT:
             return piece
     return PIECES[0]
 
@@ -64,7 +64,7 @@ def state_space(u: torch.Tensor, p: torch.Tensor, raw_col: int, dt_bias: torch.T
                  ptr(y), 0, singles, heads, groups, n, e, stream())
     if singles < S:
         check_tensor("recurrence input", u, torch.bfloat16)
-        piece = piece_tokens(batch.max_segment, heads)
+        piece = piece_tokens(T, heads)
         piece_seg, piece_tok0, pieces = batch.attention_tiles(piece, singles)
         chained = batch.max_segment > piece
         scratch = torch.empty((pieces, size), dtype=torch.float32, device=u.device) if chained else None
